@@ -17,7 +17,7 @@
 //     (the all-gather, also by peer stores) — while the tensor pipe is already working on later rounds;
 //   * a call ends when every peer has signalled that all its stores into this rank's y are performed.
 // y and the slots live in one cudaIpc-shared allocation per rank (cvllm_ipc_alloc), so `world` processes map each
-// other's buffers; a single process may also pass plain device pointers (several virtual ranks on one GPU: the tests).
+// other's buffers; a world of one may pass a plain device pointer (the tests).
 //
 // Memory model: every flag or counter that guards data read by another GPU is written after `fence.acq_rel.sys` and
 // read with `ld.acquire.sys` (csrc/allreduce.cu has the argument).  TMA stores are async-proxy writes: the storing
@@ -283,10 +283,9 @@ gemm_reduce_kernel(const __grid_constant__ GrsMaps maps, const GrsParams p) {
   } else if (warp == 1) {
     // ===================== UMMA issuer (leader CTA only) =====================
     // The whole warp walks the schedule (every value below is warp-uniform: kernel parameters, blockIdx, loop counters,
-    // the TMEM base shuffled from lane 0) and lane 0 only executes the tcgen05 instructions: the compiler then keeps
-    // addresses and descriptors on the uniform datapath.  Computed inside a one-lane region they live in vector
-    // registers and every UMMA is preceded by five R2UR moves inside an ELECT loop (21 SASS instructions per UMMA; the
-    // same finding as the prefill issuer, tools/trace_prefill.py).  A descriptor is its stage's base descriptor plus a
+    // the TMEM base shuffled from lane 0) and lane 0 only executes the tcgen05 instructions: addresses and
+    // descriptors are then uniform values for the compiler, which issues faster than the same code inside a one-lane
+    // region (the same finding as the prefill issuer, tools/trace_prefill.py).  A descriptor is its stage's base descriptor plus a
     // constant (the 14-bit start-address field cannot carry: shared memory ends below 256 KB).
     if (cr == 0) {
       constexpr uint32_t idesc = umma_idesc(BF16, 2 * kBM, kBN, false, false);

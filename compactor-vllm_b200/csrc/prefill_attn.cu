@@ -160,7 +160,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     constexpr uint32_t idesc_qk = umma_idesc(BF16, kBM, kBN, false, false);
     constexpr uint32_t idesc_pv = umma_idesc(BF16, kBM, kHD, false, true);
     const uint64_t q_desc = umma_smem_desc(smem_u32(sm.q), 16, 1024);
-    // warp-uniform copies for the issuing thread (no R2UR loop per UMMA; see prefill_attn2.cu)
+    // warp-uniform copies for the issuing thread (see prefill_attn2.cu)
     const uint32_t tmem_s0u = __shfl_sync(0xffffffffu, tmem_s0, 0), tmem_ou = tmem_s0u + 256;
 
     auto issue_pv = [&](int i) {
@@ -278,7 +278,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
 
       // ---- P = exp2(S*scale - m_ref), row sum, bf16 pack, back to TMEM ----
       const float neg_m = (m_ref == -INFINITY) ? 0.f : -m_ref;
-      // packed fp32 pairs (FFMA2 / FADD2: half the FMA-pipe issue slots of the scalar form, same roundings)
+      // packed fp32 pairs (fp32x2: half the FMA-pipe issue slots of the scalar form, same roundings)
       const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), nm2 = make_float2(neg_m, neg_m);
       float2 l2a = make_float2(0.f, 0.f), l2b = make_float2(0.f, 0.f);
 #pragma unroll

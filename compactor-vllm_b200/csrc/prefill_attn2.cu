@@ -64,15 +64,15 @@ struct Prefill2Smem {
 };
 
 // kPolyPairs = e: e of every 8 logit PAIRS take their exponentials on the FMA pipe (ex2_poly2) instead of the MUFU.
-// A warp that issues MUFU.EX2 is held for the 8 cycles its scheduler's 4-lane unit needs (59 % of a softmax warp's
-// active samples in the ncu source view); ten packed fp32x2 instructions do a PAIR.  Measured with the in-kernel trace
+// An exponential occupies its scheduler's special-function unit for 8 cycles (16 per clock and SM); a few packed fp32x2
+// operations do a PAIR on the FMA pipe instead.  Measured with the in-kernel trace
 // (cycles per KV tile, together with the converged-warp UMMA issue below, P handed over at once): e = 0: 3161, 1: 3050,
 // 2: 2881, 3: 2887, 4: 3218 — beyond a third the FMA-pipe work outweighs the MUFU time it frees.
 #ifndef CVLLM_PREFILL_POLY_PAIRS
 #define CVLLM_PREFILL_POLY_PAIRS 3
 #endif
 // P is handed to the issuer in two parts (the first kPSplit 32-key pieces, then the rest): the first PV UMMAs run while
-// the softmax group is still on the second part.  With the ELECT-loop issuer this LOST 3 % (the issuer stalled in the
+// the softmax group is still on the second part.  With the first, slower issuer this LOST 3 % (the issuer stalled in the
 // middle of a group); with the converged-warp issue it takes another 230 cycles off the tile: trace, cycles per KV tile,
 // polynomial pairs 3 of 8: split 0: 2887, 1: 2678, 2: 2647, 3: 2668 (and 3021 with 4 of 8 pairs).
 #ifndef CVLLM_PREFILL_P_SPLIT
@@ -216,9 +216,8 @@ prefill_attn2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     auto phase_of = [](int n) { return (uint32_t)((n / kSlots) & 1); };
 
     // The issuing thread is on the critical path of every hand-off (tools/trace_prefill.py: 86 cycles per UMMA in the
-    // loop against 64 on the pipe, 13 SASS instructions each).  Two things keep its per-UMMA work to a few uniform-
-    // datapath instructions: the TMEM base is made provably warp-uniform (a shuffle from lane 0: otherwise every UMMA
-    // is wrapped in an ELECT / R2UR / branch loop), and a descriptor is its tile's base descriptor plus a constant
+    // loop against 64 on the pipe).  Two things keep its per-UMMA work small (measured with that trace): the TMEM base is
+    // made provably warp-uniform (a shuffle from lane 0), and a descriptor is its tile's base descriptor plus a constant
     // (the 14-bit start-address field cannot carry: shared memory ends below 256 KB) instead of a shift and two masks.
     const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem, 0);
     auto desc_at = [](uint64_t base, uint32_t byte_off) {
@@ -385,7 +384,7 @@ prefill_attn2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         }
       };
       // P = exp2(S*scale - m_ref) packed to 16 bit over the S columns; returns the row sum of this tile.
-      // Packed fp32 pairs: one FFMA2 scales and shifts two logits, one FADD2 adds two probabilities (A/B on B200,
+      // Packed fp32 pairs: one fp32x2 FMA scales and shifts two logits, one fp32x2 add sums two probabilities (A/B on B200,
       // r02d: 7.62-7.68 ms vs 7.95-8.05 ms scalar at 32K).
       auto write_p = [&]() -> float {
         const float neg_m = (m_ref == -INFINITY) ? 0.f : -m_ref;
@@ -429,7 +428,7 @@ prefill_attn2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 
       // The row maximum of the tile is known before the first exponential.  Taking it off the critical path
       // (exponentials against the previous tiles' reference, rescale deferred by one tile) was measured on B200
-      // and changed nothing: 7.70-7.91 ms vs 7.60-7.80 ms at 32K (r02i) — the FMNMX3 chain already hides under the
+      // and changed nothing: 7.70-7.91 ms vs 7.60-7.80 ms at 32K (r02i) — the chain of maxima already hides under the
       // TMEM load latency.
       {
         const float m_new = fmaxf(m_ref, row_max());

@@ -68,14 +68,14 @@ __device__ __forceinline__ uint4 pack8(const float* x) {
 
 // packed fp32 pairs (FMUL2 / FADD2 / FFMA2 of sm_100): half the issue slots of the scalar forms, each
 // lane still rounded to nearest, and the _rn intrinsics are never contracted into an FMA
-// explicit .rn PTX: ptxas never fuses a mul.rn with an add.rn (the sm_100_rt intrinsics were seen contracted)
+// explicit .rn PTX: ptxas never fuses a mul.rn with an add.rn (the intrinsics gave fused results)
 __device__ __forceinline__ float2 mul2_rn(float2 a, float2 b) {
   uint64_t d;
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(*reinterpret_cast<uint64_t*>(&a)), "l"(*reinterpret_cast<uint64_t*>(&b)));
   return *reinterpret_cast<float2*>(&d);
 }
-// a + b as fma(a, ones, b) with `ones` = (1, 1) from a kernel parameter: ptxas contracts mul.rn.f32x2 +
-// add.rn.f32x2 into one FFMA2 (seen in SASS even with -fmad=false), which would drop the reference's rounding
+// a + b as fma(a, ones, b) with `ones` = (1, 1) from a kernel parameter: a mul.rn.f32x2
+// followed by an add.rn.f32x2 gave the bits of one fused operation (even with -fmad=false), which drops the reference's rounding
 // of the products; it cannot fold an fma whose multiplier it does not know.  a*1+b rounds once: exact.
 __device__ __forceinline__ float2 add2_rn(float2 a, float2 b, float2 ones) {
   uint64_t d;

@@ -144,7 +144,7 @@ chunk_scores_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
     // ============================ UMMA issuer ============================
     asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kRegsOther));
     constexpr uint32_t idesc = umma_idesc(BF16, kTile, kTile, false, false);
-    const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem, 0);  // warp-uniform for the compiler: no R2UR per UMMA
+    const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem, 0);  // provably warp-uniform for the compiler
     int it = 0, qn = 0;  // qn doubles as the CTA-local tile counter: TMEM buffer qn % 4
     for (int idx = next_valid(blockIdx.x); idx < total; idx = next_valid(idx + gridDim.x), ++it) {
       const int kb = it % kKBufs;

@@ -136,7 +136,7 @@ snap_umma_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant
     // ============================ UMMA issuer ============================
     asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(kRegsOther));
     constexpr uint32_t idesc = umma_idesc(BF16, kTile, kTile, false, false);
-    const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem, 0);  // warp-uniform for the compiler: no R2UR per UMMA
+    const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem, 0);  // provably warp-uniform for the compiler
     mbar_wait(&sm.q_full, 0);
     for (int t = 0; t < n_tiles; ++t) {
       const int slot = t % kSlots, buf = t & 3;

@@ -201,9 +201,8 @@ prefill_attn2_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     auto phase_of = [](int n) { return (uint32_t)((n / kSlots) & 1); };
 
     // The issuing thread is on the critical path of every hand-off (tools/trace_prefill.py: 86 cycles per UMMA in the
-    // loop against 64 on the pipe, 13 SASS instructions each).  Two things keep its per-UMMA work to a few uniform-
-    // datapath instructions: the TMEM base is made provably warp-uniform (a shuffle from lane 0: otherwise every UMMA
-    // is wrapped in an ELECT / R2UR / branch loop), and a descriptor is its tile's base descriptor plus a constant
+    // loop against 64 on the pipe).  Two things keep its per-UMMA work small (measured with that trace): the TMEM base is
+    // made provably warp-uniform (a shuffle from lane 0), and a descriptor is its tile's base descriptor plus a constant
     // (the 14-bit start-address field cannot carry: shared memory ends below 256 KB) instead of a shift and two masks.
     const uint32_t tmem_u = __shfl_sync(0xffffffffu, tmem, 0);
     auto desc_at = [](uint64_t base, uint32_t byte_off) {
