@@ -176,8 +176,9 @@ class PeerGemmAllReduce:
 
     @staticmethod
     def virtual_ranks(world: int, max_rows: int, out_features: int, device: torch.device):
-        """`world` ranks inside this process on ONE device (their kernels run side by side on `world` streams, each on
-        1/world of the SMs — set the `grs_pairs` test option accordingly).  Returns (ranks, free)."""
+        """A world of one rank inside this process on ONE device (tests, timing of the GEMM half).  Ranks of a larger
+        world wait on one another and need a GPU each.  Returns (ranks, free)."""
+        assert world == 1, "ranks whose kernels wait on one another need one GPU each"
         lib = N.lib()
         cap = int(lib.cvllm_gemm_allreduce_payload_bytes(max_rows, out_features, world))
         bases = []
