@@ -85,6 +85,8 @@ _SIGNATURES = {
     "cvllm_latent_norm_store": (_i, [_p, _i64, _i, _i, _i, _i, _i, _p, _p, _f, _p, _p, _p, _p, _p, _p, _i64, _i, _p,
                                      _i, _i, _i, _p]),
     "cvllm_latent_q_rope": (_i, [_p, _i64, _i, _i, _i, _p, _p, _p, _i64, _i, _i, _i, _i, _p]),
+    "cvllm_latent_prepare": (_i, [_p, _i64, _i, _i, _i, _i, _i, _i, _p, _f, _p, _f, _i, _p, _p, _p, _i64, _i, _i, _p, _p,
+                                  _i64, _i, _p, _i, _i, _i, _p]),
     "cvllm_sigmoid_gate": (_i, [_p, _i64, _p, _i64, _p, _i64, _i64, _i, _i, _p]),
     "cvllm_causal_conv": (_i, [_p, _i64, _i, _i, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _p, _i64, _i, _p]),
     "cvllm_conv_state_update": (_i, [_p, _i64, _i, _i, _i, _p, _p, _p, _p, _p, _i, _i, _i, _p]),
@@ -101,14 +103,15 @@ _SIGNATURES = {
     "cvllm_bias_attn_decode": (_i, [_p, _p, _p, _p, _i64, _i64, _i, _p, _p, _p, _i, _i, _p, _f, _p,
                                     _i, _i, _i, _i, _i, _i, _i, _p, _sz, _i64, _i, _p]),
     "cvllm_residual_norm": (_i, [_p, _i64, _p, _i64, _i, _p, _i64, _p, _i64, _p, _p, _p, _i64, _i, _i, _i, _f, _i, _p]),
+    "cvllm_embed_norm": (_i, [_p, _p, _i, _p, _p, _i, _p, _i64, _p, _i64, _i, _i, _i, _f, _p]),
     "cvllm_pair_hash_embed": (_i, [_p, _p, _p, _p, _p, _i64, _i64, _i64, _p, _p, _i64, _i, _i, _i, _i, _p]),
     "cvllm_token_shift_mix": (_i, [_p, _i64, _p, _i, _i, _p, _p, _p, _p, _p, _i, _i, _p, _i64, _i, _i, _p]),
     "cvllm_delta_rule": (_i, [_p, _i64, _p, _i64, _i, _i, _p, _p, _p, _p, _i64, _i, _p, _i, _f, _p, _p, _p, _p, _i, _i,
                               _p, _i64, _i, _i, _i, _i, _i, _i, _p]),
-    "cvllm_bias_attn_varlen_dist": (_i, [_p, _p, _p, _p, _i64, _i64, _i, _p, _p, _p, _p, _i, _i, _p, _i, _i, _p, _f, _p,
-                                         _i, _i, _i, _i, _i, _i, _i, _i64, _i, _i64, _i, _p]),
-    "cvllm_bias_attn_decode_dist": (_i, [_p, _p, _p, _p, _i64, _i64, _i, _p, _p, _p, _i, _i, _p, _i, _i, _p, _f, _p,
-                                         _i, _i, _i, _i, _i, _i, _i, _p, _sz, _i64, _i, _p]),
+    "cvllm_bias_attn_varlen_dist": (_i, [_p, _p, _p, _p, _i64, _i64, _i, _p, _p, _p, _p, _i, _i, _i, _p, _i, _i, _p, _f,
+                                         _p, _i64, _i, _i, _i, _i, _i, _i, _i, _i64, _i, _i64, _i, _p]),
+    "cvllm_bias_attn_decode_dist": (_i, [_p, _p, _p, _p, _i64, _i64, _i, _p, _p, _p, _i, _i, _i, _p, _i, _i, _p, _f, _p,
+                                         _i64, _i, _i, _i, _i, _i, _i, _i, _p, _sz, _i64, _i, _p]),
     "cvllm_general_delta": (_i, [_p, _i64, _i, _i, _i, _i, _p, _i64, _p, _f, _p, _i, _i, _p, _i, _f, _p, _p, _p, _p,
                                  _i, _i, _p, _i64, _i, _i, _i, _i, _p]),
     "cvllm_matrix_memory": (_i, [_p, _i64, _i, _i, _i, _i, _i, _f, _f, _p, _p, _p, _i, _i, _p, _i, _f, _p, _p, _p, _p,

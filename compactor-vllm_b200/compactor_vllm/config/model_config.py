@@ -615,8 +615,136 @@ class NununexConfig:
         return max([a.dim for a in self._attn()] or [1])
 
 
+@dataclass
+class KeptWindowAttentionConfig:
+    """Grouped-query attention without rotation: RMS norms with a weight on q and k, every value divided by its root mean
+    square, a sliding window of `window` positions (0 = none) beside which the sequence's first `keep_first` positions
+    stay visible."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0
+    keep_first: int = 0
+
+    @classmethod
+    def from_json(cls, m: dict) -> "KeptWindowAttentionConfig":
+        dim, mask = int(m["dim"]), m.get("mask") or {}
+        c = cls(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=dim,
+                vdim=int(m.get("vdim", dim)), scale=float(m.get("scale", dim ** -0.5)),
+                window=int(mask.get("size", 0) or 0), keep_first=int(mask.get("keep_first", 0) or 0))
+        if c.heads % c.kv_heads or c.window < 0 or c.keep_first < 0:
+            raise ValueError(f"attention: {c.heads} heads / {c.kv_heads} kv heads, window {c.window}, "
+                             f"first {c.keep_first} kept")
+        return c
+
+
+@dataclass
+class DirectLatentAttentionConfig:
+    """Latent attention without a query latent (layers/latent_attention.py `DirectLatentAttention`): sizes as in
+    `LatentAttentionConfig`, neighbouring pairs rotated with frequencies that may be stretched (`rot_scaling` =
+    (factor, original, fast, slow), see `yarn_rotation_frequencies`), a sliding window of `window` positions (0 = none)
+    and a learned softmax sink per head."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rot_base: float
+    rot_scaling: Optional[Tuple[float, float, float, float]] = None
+    window: int = 0
+
+    @classmethod
+    def from_json(cls, m: dict) -> "DirectLatentAttentionConfig":
+        rot = m.get("rot") or {}
+        rot_dim = int(m.get("rot_dim", rot.get("dims", 0)))
+        if int(rot.get("dims", rot_dim)) != rot_dim or rot_dim % 2:
+            raise ValueError(f"latent attention rotates its whole rotated part, an even number: rot_dim {rot_dim}, "
+                             f"rot.dims {rot.get('dims')}")
+        dim, sc = int(m["dim"]), rot.get("scaling")
+        c = cls(heads=int(m["heads"]), dim=dim, rot_dim=rot_dim, vdim=int(m.get("vdim", dim)), kv_rank=int(m["kv_rank"]),
+                scale=float(m.get("scale", (dim + rot_dim) ** -0.5)), rot_base=float(rot.get("base", 10000.0)),
+                rot_scaling=None if not sc else (float(sc["factor"]), float(sc["original"]), float(sc["fast"]),
+                                                 float(sc["slow"])),
+                window=int((m.get("mask") or {}).get("size", 0) or 0))
+        if c.window < 0:
+            raise ValueError(f"latent attention: window {c.window}")
+        return c
+
+
+@dataclass
+class PekasunLayerConfig:
+    mixer_type: str                     # "attention" | "latent_attention"
+    mixer: Any                          # KeptWindowAttentionConfig | DirectLatentAttentionConfig
+    mlp: Optional[FeedForwardConfig]    # dense, or None
+    owner: int                          # the layer whose weights this one uses (its own index as a rule)
+
+
+@dataclass
+class PekasunConfig:
+    """config.json of a Pekasun model: `vocab`, `width`, `norm.eps`, `layers` (each with `type`, `mixer`, `mlp`, and
+    `weights_of` for a layer that uses an other layer's weights with a cache of its own).  Every layer is
+    x += mixer(h) + ff(h) with h = rms_norm(x) times ONE number; the normed embedding starts the stream."""
+    vocab_size: int
+    hidden_size: int
+    rms_norm_eps: float
+    layers: List[PekasunLayerConfig]
+    torch_dtype: Any = torch.bfloat16
+    max_position_embeddings: int = 1 << 30      # rotation angles are computed from the position: no table to outgrow
+    model_type: str = "pekasun"
+    tie_word_embeddings: bool = False
+    raw: dict = field(default_factory=dict, repr=False)
+
+    MIXERS = {"attention": KeptWindowAttentionConfig, "latent_attention": DirectLatentAttentionConfig}
+
+    @classmethod
+    def from_json(cls, c: dict) -> "PekasunConfig":
+        entries, layers = c["layers"], []
+        for i, entry in enumerate(entries):
+            kind = entry["type"]
+            if kind not in cls.MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            ff = entry.get("mlp")
+            if ff is not None and ff.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: feed-forward kind {ff.get('kind')!r} is not part of this design")
+            owner, seen = i, {i}
+            while entries[owner].get("weights_of") is not None:
+                owner = int(entries[owner]["weights_of"])
+                if not 0 <= owner < len(entries) or owner in seen:
+                    raise ValueError(f"layer {i}: weights_of does not lead to a layer with weights of its own")
+                seen.add(owner)
+            mixer, mlp = cls.MIXERS[kind].from_json(entry["mixer"]), FeedForwardConfig.from_json(ff)
+            o = entries[owner]
+            if owner != i and (o["type"] != kind or cls.MIXERS[kind].from_json(o["mixer"]) != mixer
+                               or FeedForwardConfig.from_json(o.get("mlp")) != mlp):
+                raise ValueError(f"layer {i} uses the weights of layer {owner}, whose entry differs")
+            layers.append(PekasunLayerConfig(kind, mixer, mlp, owner))
+        return cls(vocab_size=int(c["vocab"]), hidden_size=int(c["width"]),
+                   rms_norm_eps=float((c.get("norm") or {}).get("eps", 1e-6)), layers=layers, raw=c)
+
+    # ---- the names the cache manager and the runner read from an HF config --------------------------
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def num_key_value_heads(self) -> int:
+        return max([l.mixer.kv_heads for l in self.layers if l.mixer_type == "attention"] or [1])
+
+    @property
+    def num_attention_heads(self) -> int:
+        return max([l.mixer.heads for l in self.layers] or [1])
+
+    @property
+    def head_dim(self) -> int:
+        return max([l.mixer.dim if l.mixer_type == "attention" else l.mixer.kv_rank + l.mixer.rot_dim
+                    for l in self.layers] or [1])
+
+
 ARCHITECTURES = {"Movolorn": MovolornConfig, "Batasun": BatasunConfig, "Fafelix": FafelixConfig,
-                 "Nununex": NununexConfig}
+                 "Nununex": NununexConfig, "Pekasun": PekasunConfig}
 
 
 def load_model_config(path: str):

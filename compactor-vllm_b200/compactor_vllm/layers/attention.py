@@ -6,6 +6,7 @@ pairs) on STORE_STREAM concurrently with causal attention over
 (b, h), then split-KV paged attention.  The KV-cache manager injects k_cache,
 v_cache, page_table, bh_seq_lens and page_size (core/memory_manager.py).
 """
+import copy
 from typing import Optional
 
 import torch
@@ -135,6 +136,34 @@ def pair_rotation_frequencies(dims: int, base: float, scaling: Optional[tuple] =
     return torch.tensor(out, dtype=torch.float64)
 
 
+def yarn_rotation_frequencies(dims: int, base: float, factor: float, original: float, fast: float,
+                              slow: float) -> torch.Tensor:
+    """Rotation frequencies stretched by YaRN (Peng et al., "YaRN: Efficient Context Window Extension of Large Language
+    Models"), dims / 2 64-bit floats.  Pair i makes original * f_i / (2 pi) turns over the original context; pairs with
+    more than `fast` turns keep f_i = base ** (-2 i / dims), pairs with fewer than `slow` get f_i / factor, and between
+    the two (whole) pair indices the weights of both change linearly.  Sine and cosine go with `yarn_amplitude`."""
+    import math
+
+    def pair_of(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo = max(math.floor(pair_of(fast)), 0)
+    hi = min(math.ceil(pair_of(slow)), dims - 1)
+    out = []
+    for i in range(dims // 2):
+        f = float(base) ** (-2.0 * i / dims)
+        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(f / factor * ramp + f * (1.0 - ramp))
+    return torch.tensor(out, dtype=torch.float64)
+
+
+def yarn_amplitude(factor: float) -> float:
+    """The factor on sine and cosine that goes with a context stretched by `factor`."""
+    import math
+
+    return 0.1 * math.log(factor) + 1.0
+
+
 def distance_buckets(rows: int, far: int, length: int) -> list:
     """Row of a learned distance-bias table of `rows` rows for the distances 0 .. length - 1: distances below
     rows // 2 have a row each, larger ones share logarithmic buckets that reach the last row at distance `far`:
@@ -164,8 +193,9 @@ class BiasedChunkAttention(nn.Module):
     `sink` False = plain softmax; `learned_sink` gives every head its own sink score (a parameter, not scaled; without
     it the score is 0).  `rotation` (inv_freq [rot_dims / 2] float64, see `pair_rotation_frequencies`) turns
     neighbouring pairs (2 i, 2 i + 1) of the first rot_dims numbers of every q and k head by position * inv_freq[i]
-    BEFORE the norm; `norm` False leaves q and k unnormed.  `window` > 0: a query sees only the keys at distances
-    0 .. window - 1.  `bucket_bias` = (rows, far): a learned table `rel` [rows, H] adds rel[bucket(i - j), h] to the
+    BEFORE the norm; `norm` False leaves q and k unnormed.  `value_norm`: every value head is stored divided by its root
+    mean square.  `window` > 0: a query sees only the keys at distances 0 .. window - 1, and - `keep_first` > 0 - the
+    sequence's first keep_first positions whatever their distance.  `bucket_bias` = (rows, far): a learned table `rel` [rows, H] adds rel[bucket(i - j), h] to the
     score (unscaled; buckets as in `distance_buckets`); the kernels read it spread out per distance (`dist_bias`,
     rebuilt by `refresh_distance_bias()` whenever `rel` changes).  forward() takes the packed projection rows
     [T, H*D + G*D + G*Dv] (row stride free): one launch rotates / norms q / k
@@ -178,10 +208,10 @@ class BiasedChunkAttention(nn.Module):
                  slopes: Optional[torch.Tensor] = None, chunk: int = 0, sink: bool = False, qk_norm: bool = False,
                  eps: float = 1e-6, values_in_keys: bool = False, learned_sink: bool = False,
                  rotation: Optional[torch.Tensor] = None, norm: bool = True, window: int = 0,
-                 bucket_bias: Optional[tuple] = None):
+                 bucket_bias: Optional[tuple] = None, keep_first: int = 0, value_norm: bool = False):
         super().__init__()
-        self.norm = bool(norm)
-        self.window = int(window)
+        self.norm, self.value_norm = bool(norm), bool(value_norm)
+        self.window, self.keep_first = int(window), int(keep_first)
         self.bias_far = 0
         self.rel = None
         if bucket_bias is not None:
@@ -205,6 +235,12 @@ class BiasedChunkAttention(nn.Module):
         self.page_table: Optional[torch.Tensor] = None
         self.bh_seq_lens: Optional[torch.Tensor] = None
         self.page_size: Optional[int] = None
+
+    def twin(self) -> "BiasedChunkAttention":
+        """Another run of the same layer: the parameters and constants are shared, the cache views are its own."""
+        other = copy.copy(self)
+        other.k_cache = other.v_cache = other.page_table = other.bh_seq_lens = other.page_size = None
+        return other
 
     @torch.no_grad()
     def refresh_distance_bias(self, rel: Optional[torch.Tensor] = None) -> None:
@@ -233,12 +269,13 @@ class BiasedChunkAttention(nn.Module):
         keys = min(max_keys, self.chunk) if self.chunk else max_keys
         if self.window:
             keys = min(keys, self.window)
+        keys = min(keys + self.keep_first, max_keys)
         ctas = max(batch * self.num_kv_heads * -(-(self.num_heads // self.num_kv_heads) // 4), 1)
         one_wave = min(296 // ctas, keys // 128)
         several = min(2048 // ctas, keys // 1024)
         return int(max(1, min(max(one_wave, several), 64)))
 
-    def forward(self, qkv: torch.Tensor) -> torch.Tensor:
+    def forward(self, qkv: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         from compactor_vllm import _native as N
 
         ctx: Context = get_context()
@@ -252,16 +289,17 @@ class BiasedChunkAttention(nn.Module):
         table = (N.ptr(pt), pt.stride(0), pt.stride(1), int(self.page_size))
         rot = self.inv_freq
         N.check(lib.cvllm_rope_qknorm_store(
-            N.ptr(qkv), qkv.stride(0), N.ptr(rot), 0 if rot is None else 2 * rot.numel(), int(self.norm),
+            N.ptr(qkv), qkv.stride(0), N.ptr(rot), 0 if rot is None else 2 * rot.numel(),
+            int(self.norm) + 2 * int(self.value_norm),
             N.ptr(self.q_norm_weight), N.ptr(self.k_norm_weight), self.eps,
             N.ptr(ctx.positions_i32), N.ptr(ctx.token_slot), N.ptr(q), N.ptr(self.k_cache), N.ptr(self.v_cache),
             *table, N.ptr(self.bh_seq_lens), T, H, G, D, Dv, RESERVED_BATCH, code, N.stream(dev)),
             "cvllm_rope_qknorm_store")
-        return self.attend(q)
+        return self.attend(q, out=out)
 
-    def attend(self, q: torch.Tensor, flat: bool = True) -> torch.Tensor:
+    def attend(self, q: torch.Tensor, flat: bool = True, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """q [T, H, D] (normed / rotated already, the step's keys in the cache) -> [T, H * Dv], or with flat=False
-        [T, H, Dv] (possibly a view of wider rows)."""
+        [T, H, Dv] (possibly a view of wider rows).  `out` [T, H * Dv] (row stride free): where to write."""
         from compactor_vllm import _native as N
 
         ctx: Context = get_context()
@@ -273,24 +311,29 @@ class BiasedChunkAttention(nn.Module):
         table = (N.ptr(pt), pt.stride(0), pt.stride(1), int(self.page_size))
         v_cache, v_stride = (self.k_cache, D) if self.values_in_keys else (self.v_cache, Dv)
         keep = Dv
-        if (self.values_in_keys and ctx.is_prefill and q.dtype == torch.bfloat16 and D == 128 and Dv < D
+        if (out is None and self.values_in_keys and ctx.is_prefill and q.dtype == torch.bfloat16 and D == 128 and Dv < D
                 and self.page_size % 128 == 0 and (H // G) % 2 == 0):
             # Values that are columns of 128-wide key rows: taking the WHOLE row as the value costs a few more
             # products and puts the portion on the tcgen05 pipeline (which serves D = Dv = 128); the columns past
             # the values are dropped on return.
             Dv = D
-        out = torch.empty((T, H, Dv), dtype=q.dtype, device=dev)
+        o_stride = H * Dv
+        if out is None:
+            out = torch.empty((T, H * Dv), dtype=q.dtype, device=dev)
+        else:
+            assert out.shape == (T, H * Dv) and out.stride(1) == 1 and out.dtype == q.dtype
+            o_stride = out.stride(0)
         if self.rel is not None and self.dist_bias is None:
             self.refresh_distance_bias()
         db = self.dist_bias
-        dist = (self.window, N.ptr(db), 0 if db is None else db.shape[0])
+        dist = (self.window, self.keep_first, N.ptr(db), 0 if db is None else db.shape[0])
         if ctx.is_prefill:
             B = ctx.batch_mapping.numel()
             N.check(lib.cvllm_bias_attn_varlen_dist(
                 N.ptr(q), N.ptr(self.k_cache), N.ptr(v_cache), *table, N.ptr(ctx.cu_seqlens_q),
                 N.ptr(ctx.seq_start), N.ptr(ctx.batch_mapping), N.ptr(self.slopes), self.chunk, *dist, int(self.sink),
-                N.ptr(self.sink_logits), self.scale, N.ptr(out), B, int(ctx.max_seqlen_q), H, G, D, Dv, T, self.k_cache.shape[0], pt.shape[-1],
-                v_stride, code, N.stream(dev)), "cvllm_bias_attn_varlen")
+                N.ptr(self.sink_logits), self.scale, N.ptr(out), o_stride, B, int(ctx.max_seqlen_q), H, G, D, Dv, T,
+                self.k_cache.shape[0], pt.shape[-1], v_stride, code, N.stream(dev)), "cvllm_bias_attn_varlen")
         else:
             assert ctx.batch_mapping.numel() == T
             splits = self.decode_splits(T, int(ctx.max_seqlen_k))
@@ -298,9 +341,9 @@ class BiasedChunkAttention(nn.Module):
             N.check(lib.cvllm_bias_attn_decode_dist(
                 N.ptr(q), N.ptr(self.k_cache), N.ptr(v_cache), *table, N.ptr(ctx.positions_i32),
                 N.ptr(ctx.batch_mapping), N.ptr(self.slopes), self.chunk, *dist, int(self.sink), N.ptr(self.sink_logits),
-                self.scale, N.ptr(out), T, H, G, D, Dv, RESERVED_BATCH, splits, N.ptr(ws), ws.numel() if ws is not None else 0, v_stride, code,
+                self.scale, N.ptr(out), o_stride, T, H, G, D, Dv, RESERVED_BATCH, splits, N.ptr(ws), ws.numel() if ws is not None else 0, v_stride, code,
                 N.stream(dev)), "cvllm_bias_attn_decode")
         if keep != Dv:
-            out = out[:, :, :keep]
+            out = out.view(T, H, Dv)[:, :, :keep]
             return out.reshape(T, H * keep) if flat else out
-        return out.view(T, H * Dv) if flat else out
+        return out if flat else out.unflatten(1, (H, Dv))

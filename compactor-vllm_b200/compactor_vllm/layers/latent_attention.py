@@ -13,6 +13,9 @@ multiplied by sigmoid(W_g h) before the output projection.
 A layer built with `source` (another LatentAttention) makes no latent of its own: it attends over the source layer's
 cache rows - written earlier in the same step - with its own queries, W_uk, W_uv, gate and output projection.
 
+`DirectLatentAttention` is the form without a query latent for layers that project their input in one product of their
+own, with a sliding window, learned sinks and a choice of rotation.
+
 Kernels: csrc/latent_attn.cu (norms + rotation + cache write; query rotation; gate) and csrc/bias_attn.cu.
 """
 from __future__ import annotations
@@ -33,14 +36,83 @@ def rotation_frequencies(rot_dim: int, base: float) -> torch.Tensor:
     return torch.tensor([float(base) ** (-2.0 * i / rot_dim) for i in range(rot_dim // 2)], dtype=torch.float64)
 
 
-def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
-    """x * sigmoid(gate), both [T, width] with unit inner stride (row strides free)."""
+def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x * sigmoid(gate), both [T, width] with unit inner stride (row strides free, also of `out` when given)."""
     T, width = x.shape
     assert gate.shape == x.shape and x.stride(1) == 1 and gate.stride(1) == 1 and gate.dtype == x.dtype
-    out = torch.empty((T, width), dtype=x.dtype, device=x.device)
+    if out is None:
+        out = torch.empty((T, width), dtype=x.dtype, device=x.device)
+    assert out.shape == x.shape and out.stride(1) == 1 and out.dtype == x.dtype
     N.check(N.lib().cvllm_sigmoid_gate(N.ptr(x), x.stride(0), N.ptr(gate), gate.stride(0), N.ptr(out), out.stride(0), T,
                                        width, N.block_dtype_code(x.dtype), N.stream(x.device)), "cvllm_sigmoid_gate")
     return out
+
+
+def absorb_queries(q: torch.Tensor, uk: torch.Tensor, q_full: torch.Tensor) -> None:
+    """q_full[t, h, :r] = q[t, h, :dim] W_uk[h] for uk [H, dim, r]: [H, T, dim] x [H, dim, r] into the first r columns of
+    the attention's query rows."""
+    dim, r = uk.shape[1], uk.shape[2]
+    torch.bmm(q[:, :, :dim].transpose(0, 1), uk, out=q_full[:, :, :r].transpose(0, 1))
+
+
+def expand_values(o_lat: torch.Tensor, uv: torch.Tensor) -> torch.Tensor:
+    """o_lat [T, H, r] (the heads' weighted latents), uv [H, vdim, r] -> [T, H * vdim]."""
+    o = torch.empty((o_lat.shape[0], uv.shape[0], uv.shape[1]), dtype=o_lat.dtype, device=o_lat.device)
+    torch.bmm(o_lat.transpose(0, 1), uv.transpose(1, 2), out=o.transpose(0, 1))
+    return o.flatten(1)
+
+
+class DirectLatentAttention(nn.Module):
+    """Latent attention whose queries come straight from the layer's input (no query latent), for layers that bring the
+    projections of their input themselves: `forward` takes the columns [q | latent and shared key part | gate] of that
+    projection and writes the gated, concatenated heads to `out`; the output projection is the layer's as well.
+
+    Options beside `LatentAttention`'s: `window` (sliding window), `learned_sink` (one more term exp(sink_h) in every
+    head's denominator), `inv_freq` (rotation frequencies, rot_dim / 2 64-bit floats), `amplitude` (a factor on sine and
+    cosine), `neighbours` (number 2 i turns with 2 i + 1 instead of i with i + rot_dim / 2).  The cache views and the
+    sink live in `attn`, so that several runs of one layer can share the weights (`attn.twin()`)."""
+
+    def __init__(self, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float, eps: float, *,
+                 inv_freq: torch.Tensor, amplitude: float = 1.0, neighbours: bool = False, window: int = 0,
+                 learned_sink: bool = False, gate: bool = True, dtype: Optional[torch.dtype] = None):
+        super().__init__()
+        assert inv_freq.dtype == torch.float64 and 2 * inv_freq.numel() == rot_dim
+        self.heads, self.dim, self.rot_dim, self.vdim = int(heads), int(dim), int(rot_dim), int(vdim)
+        self.kv_rank, self.eps = int(kv_rank), float(eps)
+        self.amplitude, self.neighbours, self.gate = float(amplitude), bool(neighbours), bool(gate)
+        self.row = self.kv_rank + self.rot_dim     # numbers per cache row
+        self.attn = BiasedChunkAttention(self.heads, 1, self.row, self.kv_rank, scale, values_in_keys=True,
+                                         sink=learned_sink, learned_sink=learned_sink, window=window)
+        self.out_width = self.heads * self.vdim
+        self.in_parts = [("q", self.heads * (self.dim + self.rot_dim)), ("dkv", self.row)]
+        if self.gate:
+            self.in_parts.append(("g", self.out_width))
+        self.in_cols = sum(n for _, n in self.in_parts)
+        self.kv_norm = nn.Parameter(torch.ones(self.kv_rank, dtype=torch.float32))
+        self.uk = nn.Parameter(torch.empty(self.heads, self.dim, self.kv_rank, dtype=dtype))
+        self.uv = nn.Parameter(torch.empty(self.heads, self.vdim, self.kv_rank, dtype=dtype))
+        self.register_buffer("inv_freq", inv_freq.contiguous(), persistent=False)
+
+    def forward(self, cols: torch.Tensor, attn: BiasedChunkAttention, out: torch.Tensor) -> None:
+        ctx = get_context()
+        assert attn.k_cache is not None, "KV cache must be initialized"
+        assert cols.shape[1] == self.in_cols and cols.stride(1) == 1
+        T, H, D, R, r = cols.shape[0], self.heads, self.dim, self.rot_dim, self.kv_rank
+        kv_off = H * (D + R)
+        q_full = torch.empty((T, H, self.row), dtype=cols.dtype, device=cols.device)
+        pt = attn.page_table
+        N.check(N.lib().cvllm_latent_prepare(
+            N.ptr(cols), cols.stride(0), 0, H, D, kv_off, r, R, N.ptr(self.kv_norm), self.eps, N.ptr(self.inv_freq),
+            self.amplitude, int(self.neighbours), N.ptr(ctx.positions_i32), N.ptr(ctx.token_slot), N.ptr(q_full),
+            q_full.stride(0), self.row, r, N.ptr(attn.k_cache), N.ptr(pt), pt.stride(0), int(attn.page_size),
+            N.ptr(attn.bh_seq_lens), T, RESERVED_BATCH, N.block_dtype_code(cols.dtype), N.stream(cols.device)),
+            "cvllm_latent_prepare")
+        absorb_queries(cols[:, :kv_off].unflatten(1, (H, D + R)), self.uk, q_full)
+        o = expand_values(attn.attend(q_full, flat=False), self.uv)
+        if self.gate:
+            sigmoid_gate(o, cols[:, kv_off + self.row:], out)
+        else:
+            out.copy_(o)
 
 
 class LatentAttention(nn.Module):
@@ -80,7 +152,7 @@ class LatentAttention(nn.Module):
         ctx = get_context()
         attn = self._cache()
         T = h.shape[0]
-        H, D, R, Dv, r = self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank
+        H, D, R, r = self.heads, self.dim, self.rot_dim, self.kv_rank
         dev, lib, st = h.device, N.lib(), N.stream(h.device)
         proj = self.in_proj(h)
         code = N.block_dtype_code(proj.dtype)
@@ -93,11 +165,8 @@ class LatentAttention(nn.Module):
             RESERVED_BATCH, code, st), "cvllm_latent_norm_store")
         q = self.uq_proj(cq).view(T, H, D + R)
         q_full = torch.empty((T, H, self.row), dtype=proj.dtype, device=dev)
-        # q_abs[h] = q_plain[h] W_uk[h]: [H, T, D] x [H, D, r] into the first r columns of the attention's query rows
-        torch.bmm(q[:, :, :D].transpose(0, 1), self.uk, out=q_full[:, :, :r].transpose(0, 1))
+        absorb_queries(q, self.uk, q_full)
         N.check(lib.cvllm_latent_q_rope(N.ptr(q), q.stride(0), H, D, R, N.ptr(self.inv_freq), N.ptr(ctx.positions_i32),
                                         N.ptr(q_full), q_full.stride(0), self.row, r, T, code, st), "cvllm_latent_q_rope")
         o_lat = attn.attend(q_full, flat=False)           # [T, H, r], possibly a view of wider rows
-        o = torch.empty((T, H, Dv), dtype=proj.dtype, device=dev)
-        torch.bmm(o_lat.transpose(0, 1), self.uv.transpose(1, 2), out=o.transpose(0, 1))
-        return self.o_proj(sigmoid_gate(o.view(T, H * Dv), proj[:, self.g_off:]))
+        return self.o_proj(sigmoid_gate(expand_values(o_lat, self.uv), proj[:, self.g_off:]))

@@ -94,7 +94,7 @@ class NormWeight(nn.Module):
         self.weight = nn.Parameter(torch.ones(size, dtype=torch.float32))
 
 
-NORM_RMS, NORM_LAYER = 0, 1
+NORM_RMS, NORM_LAYER, NORM_RMS_ONE_GAIN = 0, 1, 2
 
 
 def residual_norm(resid: torch.Tensor, *, add: tuple = (), add_f32: torch.Tensor | None = None,
@@ -104,7 +104,8 @@ def residual_norm(resid: torch.Tensor, *, add: tuple = (), add_f32: torch.Tensor
 
         resid += add[0] + add[1] + add_f32      (up to two branch outputs in the activations' type, one fp32 tensor)
         weight given:  returns norm(resid) in `out_dtype` - NORM_LAYER: (x - mean) / sqrt(var + eps) * weight + bias,
-                       NORM_RMS: x / sqrt(mean(x^2) + eps) * weight
+                       NORM_RMS: x / sqrt(mean(x^2) + eps) * weight, NORM_RMS_ONE_GAIN: the same with a weight of one
+                       number for all coordinates
 
     i.e. the residual sum of a layer whose sublayers run side by side on one normed input, fused with the norm in
     front of the next layer.  Sum and statistics are fp32; weight and bias are fp32 tensors."""
@@ -123,6 +124,7 @@ def residual_norm(resid: torch.Tensor, *, add: tuple = (), add_f32: torch.Tensor
     out, o_code, o_stride = None, N.CVLLM_F32, 0
     if weight is not None:
         assert weight.dtype == torch.float32 and (bias is None or bias.dtype == torch.float32)
+        assert weight.numel() == (1 if kind == NORM_RMS_ONE_GAIN else width)
         out = torch.empty((rows, width), dtype=out_dtype or torch.float32, device=resid.device)
         o_code, o_stride = N.block_dtype_code(out.dtype), out.stride(0)
     rc = N.lib().cvllm_residual_norm(
@@ -131,6 +133,32 @@ def residual_norm(resid: torch.Tensor, *, add: tuple = (), add_f32: torch.Tensor
         N.ptr(bias), N.ptr(out), o_stride, o_code, rows, width, float(eps), int(kind), N.stream(resid.device))
     N.check(rc, "cvllm_residual_norm")
     return out
+
+
+def embed_norm(input_ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, *,
+               next_weight: torch.Tensor | None = None, eps: float = 1e-6, out_dtype: torch.dtype | None = None):
+    """One launch of `cvllm_embed_norm`: the normed token embedding that starts a 32-bit residual stream, and the norm in
+    front of the first layer.
+
+        resid = rms_norm(table[input_ids]) * weight                 (fp32 [T, width])
+        next_weight given:  out = rms_norm(resid) * next_weight     in `out_dtype`
+
+    The weights are fp32, [width] each or one number each.  Returns (resid, out or None)."""
+    T, width = input_ids.numel(), table.shape[1]
+    assert input_ids.dtype == torch.int64 and input_ids.is_contiguous() and table.is_contiguous()
+    one = weight.numel() == 1 and width > 1
+    for w in (weight, next_weight):
+        assert w is None or (w.dtype == torch.float32 and w.numel() == (1 if one else width))
+    resid = torch.empty((T, width), dtype=torch.float32, device=table.device)
+    out, o_code, o_stride = None, N.CVLLM_F32, 0
+    if next_weight is not None:
+        out = torch.empty((T, width), dtype=out_dtype or torch.float32, device=table.device)
+        o_code, o_stride = N.block_dtype_code(out.dtype), out.stride(0)
+    rc = N.lib().cvllm_embed_norm(
+        N.ptr(input_ids), N.ptr(table), N.block_dtype_code(table.dtype), N.ptr(weight), N.ptr(next_weight), int(one),
+        N.ptr(resid), resid.stride(0), N.ptr(out), o_stride, o_code, T, width, float(eps), N.stream(table.device))
+    N.check(rc, "cvllm_embed_norm")
+    return resid, out
 
 
 def gated_residual_norm(resid: torch.Tensor, *, branch: torch.Tensor | None = None, gate: torch.Tensor | None = None,

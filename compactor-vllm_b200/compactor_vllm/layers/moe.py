@@ -19,13 +19,17 @@ ROUTE_SOFTMAX_ALL, ROUTE_TOP_LOGITS, ROUTE_SIGMOID = 0, 1, 2
 ACT_RELU_SQUARED = 0      # kinds of `unary_act`
 
 
-def gated_act(x: torch.Tensor, kind: int, rows: int | None = None, limit: float = 0.0) -> torch.Tensor:
+def gated_act(x: torch.Tensor, kind: int, rows: int | None = None, limit: float = 0.0,
+              out: torch.Tensor | None = None) -> torch.Tensor:
     """x [T, 2F] = [gate | up] -> [T, F] (fp32 inside).  kind ACT_SILU / ACT_GELU_TANH: act(gate) * up;
     ACT_CLAMPED_GLU: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(1.702 g) * (u + 1).
-    `rows`: only the first so many rows are computed (the output still has T rows)."""
+    `rows`: only the first so many rows are computed (the output still has T rows).  `out`: where to write (row stride
+    free, e.g. a column range of a wider buffer)."""
     T, F2 = x.shape
     assert F2 % 2 == 0 and x.stride(1) == 1
-    out = torch.empty((T, F2 // 2), dtype=x.dtype, device=x.device)
+    if out is None:
+        out = torch.empty((T, F2 // 2), dtype=x.dtype, device=x.device)
+    assert out.shape == (T, F2 // 2) and out.stride(1) == 1 and out.dtype == x.dtype
     rc = N.lib().cvllm_gated_act(N.ptr(x), x.stride(0), N.ptr(out), out.stride(0), T if rows is None else int(rows),
                                  F2 // 2, int(kind), float(limit), N.block_dtype_code(x.dtype), N.stream(x.device))
     N.check(rc, "cvllm_gated_act")

@@ -6,6 +6,8 @@
 // score(i, j) = scale * q_i . k_j - slope_h * (i - j) for keys j <= i of the same chunk
 // (floor(i / chunk) == floor(j / chunk), chunk 0 = one chunk), positions counted from the start of the
 // sequence; p_j = exp(s_j) / (sink + sum_j exp(s_j)) with sink = 1 (a key of score 0 without a value) or 0.
+// Optional masks and biases beside these: a sliding window with kept first tokens, a learned bias per distance
+// (DistBias), and a learned sink score per head.
 // The new tokens' keys are in the cache before the attention launches read it, so both read keys from one place.
 // All arithmetic is fp32; 16-bit storage only rounds q, k, v and the output.
 #include "common.cuh"
@@ -49,11 +51,13 @@ inline PagedKV make_paged(const void* k, const void* v, const int32_t* table, in
 // A sliding window and a learned bias per distance, beside the linear bias and the chunk mask (all may be combined):
 // a query at position i sees the keys at distances 0 .. window - 1 (window 0: no limit), and the score of the key at
 // distance n gets table[min(n, rows - 1), h] (fp32 [rows, H]; NULL: none).  The table is made by the caller, so any
-// rule from distance to bias (buckets of a smaller learned table, for one) is served.
+// rule from distance to bias (buckets of a smaller learned table, for one) is served.  keep > 0: the sequence's first
+// `keep` positions stay visible to every later query whatever the window and the chunk say.
 struct DistBias {
   const float* table;
   int rows;
   int window;
+  int keep;
 };
 
 __device__ __forceinline__ float dist_bias_at(const DistBias& db, int n, int H, int h) {
@@ -67,6 +71,16 @@ __device__ __forceinline__ int first_key(int pi, int chunk, const DistBias& db) 
   return lo;
 }
 
+// The keys a group of queries reads, as one list of `count` entries without the gap between the kept first tokens and
+// the window: entries 0 .. kept - 1 are positions 0 .. kept - 1, later ones are positions entry + shift.  `lo` is the
+// first position the group's earliest query sees through window and chunk, `last` its last position.
+struct KeyList {
+  int kept, shift, count;
+  __device__ __forceinline__ KeyList(int lo, int last, const DistBias& db)
+      : kept(min(db.keep, lo)), shift(lo - kept), count(last + 1 - shift) {}
+  __device__ __forceinline__ int pos(int entry) const { return entry < kept ? entry : entry + shift; }
+};
+
 __device__ __forceinline__ int64_t cache_row(const PagedKV& c, int slot, int g, int pos) {
   const int lp = c.page_shift >= 0 ? pos >> c.page_shift : pos / c.page_size;
   const int page = c.table[slot * c.table_stride_slot + g * c.table_stride_head + lp];
@@ -77,7 +91,8 @@ __device__ __forceinline__ int64_t cache_row(const PagedKV& c, int slot, int g, 
 // q / k rotation + norm + store.  One CTA per token; its warps take the token's H + 2G head rows in turn.
 // Rotation (inv_freq != NULL): neighbours (2i, 2i + 1) of the first rot_dims numbers of every q and k head turn by
 // pos * inv_freq[i] (64-bit angle, fp32 sine / cosine in shared memory, once per CTA) BEFORE the norm.
-// norm 0: no norm; 1: x / sqrt(mean(x^2) + eps), times the weight when one is given.
+// norm is a bit mask: bit 0, q and k heads become x / sqrt(mean(x^2) + eps), times the weight when one is given; bit 1,
+// value heads become x / sqrt(mean(x^2) + eps) (no weight).
 // ---------------------------------------------------------------------------------------------------------
 struct Rotation {
   const double* inv_freq;   // [dims / 2] or NULL (no rotation)
@@ -136,8 +151,8 @@ __global__ void __launch_bounds__(128) qknorm_store_kernel(
         ss += a * a + b * b;
       }
       ss = warp_sum(ss);
-      const float inv = norm ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
-      const float* w = norm ? (is_q ? q_w : k_w) : nullptr;
+      const float inv = (norm & 1) ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
+      const float* w = (norm & 1) ? (is_q ? q_w : k_w) : nullptr;
       T* dst = is_q ? q_out + ((int64_t)t * H + r) * D : k_cache + cache_row(c, slot, r - H, pos) * D;
       for (int p = lane; p < pairs; p += 32) {
         float a, b;
@@ -152,7 +167,14 @@ __global__ void __launch_bounds__(128) qknorm_store_kernel(
       const int g = r - H - G;
       const T* src = row + (int64_t)(H + G) * D + (int64_t)g * Dv;
       T* dst = v_cache + cache_row(c, slot, g, pos) * Dv;
-      for (int d = lane; d < Dv; d += 32) dst[d] = src[d];
+      if (norm & 2) {
+        float ss = 0.f;
+        for (int d = lane; d < Dv; d += 32) ss += to_f<T>(src[d]) * to_f<T>(src[d]);
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)Dv + eps);
+        for (int d = lane; d < Dv; d += 32) dst[d] = from_f<T>(to_f<T>(src[d]) * inv);
+      } else {
+        for (int d = lane; d < Dv; d += 32) dst[d] = src[d];
+      }
       if (lane == 0 && bh_lens) atomicMax(bh_lens + slot * G + g, pos + 1);
     }
   }
@@ -168,7 +190,7 @@ template <typename T, int BN, int DVC>
 __global__ void __launch_bounds__(256) bias_attn_varlen_kernel(
     const T* __restrict__ q, PagedKV c, const int32_t* __restrict__ cu_q, const int32_t* __restrict__ seq_start,
     const int32_t* __restrict__ batch_mapping, const float* __restrict__ slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale,
-    T* __restrict__ out, int H, int G, int D, int Dv) {
+    T* __restrict__ out, int64_t o_stride, int H, int G, int D, int Dv) {
   constexpr int NJ = BN / 16;
   const int b = blockIdx.y, h = blockIdx.z;
   const int q0 = cu_q[b], n_new = cu_q[b + 1] - q0;
@@ -179,7 +201,7 @@ __global__ void __launch_bounds__(256) bias_attn_varlen_kernel(
   const int start = seq_start[b];
   const int rows = min(BM, n_new - tile0);
   const int p_first = start + tile0, p_last = p_first + rows - 1;
-  const int lo = first_key(p_first, chunk, db);
+  const KeyList keys(first_key(p_first, chunk, db), p_last, db);
   const float slope = slopes ? slopes[h] : 0.f;
 
   extern __shared__ float smem[];
@@ -207,10 +229,10 @@ __global__ void __launch_bounds__(256) bias_attn_varlen_kernel(
   const T* kc = static_cast<const T*>(c.k);
   const T* vc = static_cast<const T*>(c.v);
 
-  for (int k0 = lo; k0 <= p_last; k0 += BN) {
+  for (int k0 = 0; k0 < keys.count; k0 += BN) {
     __syncthreads();  // the previous tile's Ks / Vs / Ps are no longer read
-    const int nk = min(BN, p_last + 1 - k0);
-    if (tid < nk) rix[tid] = cache_row(c, slot, g, k0 + tid);
+    const int nk = min(BN, keys.count - k0);
+    if (tid < nk) rix[tid] = cache_row(c, slot, g, keys.pos(k0 + tid));
     __syncthreads();
     for (int i = tid; i < BN * D; i += 256) {
       const int r = i / D, d = i - r * D;
@@ -245,8 +267,8 @@ __global__ void __launch_bounds__(256) bias_attn_varlen_kernel(
       float mx = -INFINITY;
 #pragma unroll
       for (int j = 0; j < NJ; ++j) {
-        const int pj = k0 + tx + 16 * j;
-        const bool ok = r < rows && pj <= pi && pj >= lo_i;
+        const int pj = keys.pos(k0 + tx + 16 * j);
+        const bool ok = r < rows && pj <= pi && (pj >= lo_i || pj < db.keep);
         s[i][j] = ok ? s[i][j] * scale - slope * (float)(pi - pj) + dist_bias_at(db, pi - pj, H, h) : -INFINITY;
         mx = fmaxf(mx, s[i][j]);
       }
@@ -293,7 +315,7 @@ __global__ void __launch_bounds__(256) bias_attn_varlen_kernel(
 #pragma unroll
     for (int cc = 0; cc < DVC; ++cc) {
       const int col = tx + 16 * cc;
-      if (col < Dv) out[((int64_t)(q0 + tile0 + r) * H + h) * Dv + col] = from_f<T>(acc[i][cc] * inv);
+      if (col < Dv) out[(int64_t)(q0 + tile0 + r) * o_stride + (int64_t)h * Dv + col] = from_f<T>(acc[i][cc] * inv);
     }
   }
 }
@@ -333,7 +355,7 @@ template <int DMAX>
 __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
     const __nv_bfloat16* __restrict__ q, PagedKV c, const int32_t* __restrict__ cu_q,
     const int32_t* __restrict__ seq_start, const int32_t* __restrict__ batch_mapping,
-    const float* __restrict__ slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, __nv_bfloat16* __restrict__ out, int H, int G,
+    const float* __restrict__ slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, __nv_bfloat16* __restrict__ out, int64_t o_stride, int H, int G,
     int D, int Dv) {
   constexpr int BN = 64, LD = DMAX + 8, KS = DMAX / 16, NV = DMAX / 8;
   constexpr float kL2e = 1.4426950408889634f;   // scores in log2 units: one ex2.approx per exponential
@@ -350,7 +372,7 @@ __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
   const int g = h / (H / G);
   const int rows = min(BM, n_new - tile0);
   const int p_first = seq_start[b] + tile0, p_last = p_first + rows - 1;
-  const int lo = first_key(p_first, chunk, db);
+  const KeyList keys(first_key(p_first, chunk, db), p_last, db);
   const float slope2 = slopes ? slopes[h] * kL2e : 0.f;
   const float scale2 = scale * kL2e;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, quad = lane >> 2, tq = lane & 3;
@@ -360,20 +382,20 @@ __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
   const int kvec = D / 8, vvec = Dv / 8;
 
   auto issue_tile = [&](int stage, int k0) {
-    const int nk = min(BN, p_last + 1 - k0);
+    const int nk = min(BN, keys.count - k0);
     for (int i = tid; i < BN * kvec; i += 128) {
       const int r = i / kvec, cv = i - r * kvec;
       const bool in = r < nk;
-      cp_async16(&Ks[stage][r][cv * 8], in ? kc + cache_row(c, slot, g, k0 + r) * D + cv * 8 : kc, in ? 16 : 0);
+      cp_async16(&Ks[stage][r][cv * 8], in ? kc + cache_row(c, slot, g, keys.pos(k0 + r)) * D + cv * 8 : kc, in ? 16 : 0);
     }
     for (int i = tid; i < BN * (DMAX / 8); i += 128) {   // every column of the tile: unused ones must not hold NaN
       const int r = i / (DMAX / 8), cv = i - r * (DMAX / 8);
       const bool in = r < nk && cv < vvec;
-      cp_async16(&Vs[stage][r][cv * 8], in ? vc + cache_row(c, slot, g, k0 + r) * c.v_stride + cv * 8 : vc, in ? 16 : 0);
+      cp_async16(&Vs[stage][r][cv * 8], in ? vc + cache_row(c, slot, g, keys.pos(k0 + r)) * c.v_stride + cv * 8 : vc, in ? 16 : 0);
     }
     cp_async_commit();
   };
-  issue_tile(0, lo);
+  issue_tile(0, 0);
 
   uint32_t qa[KS][4];
 #pragma unroll
@@ -405,9 +427,9 @@ __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
   const int warp_lo = first_key(warp_first + 15, chunk, db);
 
   int stage = 0;
-  for (int k0 = lo; k0 <= p_last; k0 += BN, stage ^= 1) {
-    const int nk = min(BN, p_last + 1 - k0);
-    if (k0 + BN <= p_last) {
+  for (int k0 = 0; k0 < keys.count; k0 += BN, stage ^= 1) {
+    const int nk = min(BN, keys.count - k0);
+    if (k0 + BN < keys.count) {
       issue_tile(stage ^ 1, k0 + BN);
       cp_async_wait<1>();
     } else {
@@ -434,12 +456,13 @@ __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
       }
     }
     float mx[2] = {-INFINITY, -INFINITY};
-    if (k0 + BN - 1 <= warp_first && k0 >= warp_lo) {
+    const int p0 = k0 + keys.shift;   // position of the tile's first key when the tile has no kept first tokens
+    if (k0 >= keys.kept && p0 + BN - 1 <= warp_first && p0 >= warp_lo) {
 #pragma unroll
       for (int nb = 0; nb < BN / 8; ++nb)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int pj = k0 + nb * 8 + tq * 2 + (e & 1);
+          const int pj = p0 + nb * 8 + tq * 2 + (e & 1);
           const int dist = ((e & 2) ? pi_hi : pi_lo) - pj;
           s[nb][e] = s[nb][e] * scale2 - slope2 * (float)dist + dist_bias_at(db, dist, H, h) * kL2e;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[nb][e]);
@@ -449,10 +472,10 @@ __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
       for (int nb = 0; nb < BN / 8; ++nb)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          const int pj = k0 + nb * 8 + tq * 2 + (e & 1);
+          const int pj = keys.pos(k0 + nb * 8 + tq * 2 + (e & 1));
           const int pi = (e & 2) ? pi_hi : pi_lo;
           const int lo_i = (e & 2) ? lo_hi : lo_lo;
-          const bool ok = ((e & 2) ? r_hi : r_lo) < rows && pj <= pi && pj >= lo_i;
+          const bool ok = ((e & 2) ? r_hi : r_lo) < rows && pj <= pi && (pj >= lo_i || pj < db.keep);
           s[nb][e] = ok ? s[nb][e] * scale2 - slope2 * (float)(pi - pj) + dist_bias_at(db, pi - pj, H, h) * kL2e
                         : -INFINITY;
           mx[e >> 1] = fmaxf(mx[e >> 1], s[nb][e]);
@@ -516,10 +539,10 @@ __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
     const int col = nb * 8 + tq * 2;
     if (col < Dv) {
       if (r_lo < rows)
-        *reinterpret_cast<uint32_t*>(out + ((int64_t)(q0 + tile0 + r_lo) * H + h) * Dv + col) =
+        *reinterpret_cast<uint32_t*>(out + (int64_t)(q0 + tile0 + r_lo) * o_stride + (int64_t)h * Dv + col) =
             pack2<true>(o[nb][0] * inv[0], o[nb][1] * inv[0]);
       if (r_hi < rows)
-        *reinterpret_cast<uint32_t*>(out + ((int64_t)(q0 + tile0 + r_hi) * H + h) * Dv + col) =
+        *reinterpret_cast<uint32_t*>(out + (int64_t)(q0 + tile0 + r_hi) * o_stride + (int64_t)h * Dv + col) =
             pack2<true>(o[nb][2] * inv[1], o[nb][3] * inv[1]);
     }
   }
@@ -527,15 +550,15 @@ __global__ void __launch_bounds__(128) bias_attn_varlen_mma_kernel(
 
 template <int DMAX>
 int launch_varlen_mma(const void* q, const PagedKV& c, const int32_t* cu_q, const int32_t* seq_start, const int32_t* bm,
-                      const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out, int B, int max_new, int H,
-                      int G, int D, int Dv, cudaStream_t st) {
+                      const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out, int64_t o_stride, int B, int max_new,
+                      int H, int G, int D, int Dv, cudaStream_t st) {
   static std::atomic<uint64_t> mask{0};
   const int smem = 4 * 64 * (DMAX + 8) * 2;
   auto kern = bias_attn_varlen_mma_kernel<DMAX>;
   CVLLM_CHECK_CUDA(ensure_max_dyn_smem(reinterpret_cast<const void*>(kern), smem, mask));
   dim3 grid(cdiv(max_new, BM), B, H);
   kern<<<grid, 128, smem, st>>>(static_cast<const __nv_bfloat16*>(q), c, cu_q, seq_start, bm, slopes, chunk, db, sink, sink_logits,
-                                scale, static_cast<__nv_bfloat16*>(out), H, G, D, Dv);
+                                scale, static_cast<__nv_bfloat16*>(out), o_stride, H, G, D, Dv);
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }
@@ -552,21 +575,21 @@ template <typename T>
 __global__ void __launch_bounds__(kDecWarps * 32) bias_attn_decode_kernel(
     const T* __restrict__ q, PagedKV c, const int32_t* __restrict__ positions,
     const int32_t* __restrict__ batch_mapping, const float* __restrict__ slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale,
-    T* __restrict__ out, int H, int G, int D, int Dv, int reserved_slot) {
+    T* __restrict__ out, int64_t o_stride, int H, int G, int D, int Dv, int reserved_slot) {
   extern __shared__ float smem[];
   float* qs = smem;                         // [D]
   float* part = qs + D;                     // [kDecWarps][2 + Dv]
   const int b = blockIdx.x, h = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int slot = batch_mapping[b];
-  T* o = out + ((int64_t)b * H + h) * Dv;
+  T* o = out + (int64_t)b * o_stride + (int64_t)h * Dv;
   if (slot == reserved_slot) {
     for (int d = threadIdx.x; d < Dv; d += blockDim.x) o[d] = from_f<T>(0.f);
     return;
   }
   const int g = h / (H / G);
   const int pi = positions[b];
-  const int lo = first_key(pi, chunk, db);
+  const KeyList keys(first_key(pi, chunk, db), pi, db);
   const float slope = slopes ? slopes[h] : 0.f;
   for (int d = threadIdx.x; d < D; d += blockDim.x) qs[d] = to_f<T>(q[((int64_t)b * H + h) * D + d]);
   __syncthreads();
@@ -575,9 +598,9 @@ __global__ void __launch_bounds__(kDecWarps * 32) bias_attn_decode_kernel(
   float m = -INFINITY, l = 0.f, acc[kDecCols];
 #pragma unroll
   for (int cc = 0; cc < kDecCols; ++cc) acc[cc] = 0.f;
-  for (int k0 = lo + warp * 32; k0 <= pi; k0 += kDecWarps * 32) {
-    const int pj = k0 + lane;
-    const bool ok = pj <= pi;
+  for (int k0 = warp * 32; k0 < keys.count; k0 += kDecWarps * 32) {
+    const int pj = keys.pos(k0 + lane);
+    const bool ok = k0 + lane < keys.count;
     const int64_t row = ok ? cache_row(c, slot, g, pj) : 0;
     float s = -INFINITY;
     if (ok) {
@@ -593,7 +616,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) bias_attn_decode_kernel(
     m = m_new;
 #pragma unroll
     for (int cc = 0; cc < kDecCols; ++cc) acc[cc] *= corr;
-    const int nk = min(32, pi + 1 - k0);
+    const int nk = min(32, keys.count - k0);
     for (int j = 0; j < nk; ++j) {
       const float pj_w = __shfl_sync(0xffffffffu, p, j);
       const int64_t rj = __shfl_sync(0xffffffffu, row, j);
@@ -709,6 +732,7 @@ __global__ void __launch_bounds__(128) qknorm_store_vec_kernel(
   const bool stores = slot != reserved_slot;
   float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
   if ((is_q || (is_k && stores)) && cb < D) load8<T>(row + (int64_t)r * D + cb, x);
+  if (is_v && stores && cb < Dv) load8<T>(row + (int64_t)(H + G) * D + (int64_t)(r - H - G) * Dv + cb, x);
   if (half > 0 && (is_q || is_k)) {   // the lane's four pairs of neighbours
 #pragma unroll
     for (int e = 0; e < 8; e += 2) {
@@ -725,8 +749,8 @@ __global__ void __launch_bounds__(128) qknorm_store_vec_kernel(
   for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
   for (int o = lpr >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);   // every lane takes part
   if ((is_q || (is_k && stores)) && cb < D) {
-    const float inv = norm ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
-    const float* w = norm ? (is_q ? q_w : k_w) : nullptr;
+    const float inv = (norm & 1) ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
+    const float* w = (norm & 1) ? (is_q ? q_w : k_w) : nullptr;
 #pragma unroll
     for (int e = 0; e < 8; ++e) x[e] = w ? x[e] * inv * w[cb + e] : x[e] * inv;
     T* dst = is_q ? q_out + ((int64_t)t * H + r) * D : k_cache + cache_row(c, slot, r - H, pos) * D;
@@ -735,9 +759,12 @@ __global__ void __launch_bounds__(128) qknorm_store_vec_kernel(
   if (is_v && stores) {
     const int g = r - H - G;
     if (cb < Dv) {
-      float v[8];
-      load8<T>(row + (int64_t)(H + G) * D + (int64_t)g * Dv + cb, v);
-      store8<T>(v_cache + cache_row(c, slot, g, pos) * Dv + cb, v);
+      if (norm & 2) {
+        const float inv = 1.0f / sqrtf(ss / (float)Dv + eps);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] *= inv;
+      }
+      store8<T>(v_cache + cache_row(c, slot, g, pos) * Dv + cb, x);
     }
     if (cb == 0 && bh_lens) atomicMax(bh_lens + slot * G + g, pos + 1);
   }
@@ -747,7 +774,8 @@ template <typename T, int CH>
 __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
     const T* __restrict__ q, PagedKV c, const int32_t* __restrict__ positions,
     const int32_t* __restrict__ batch_mapping, const float* __restrict__ slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale,
-    T* __restrict__ out, float* __restrict__ part, int H, int G, int D, int Dv, int splits, int reserved_slot) {
+    T* __restrict__ out, int64_t o_stride, float* __restrict__ part, int H, int G, int D, int Dv, int splits,
+    int reserved_slot) {
   __shared__ float qs[kDecTile][64 * CH];
   __shared__ float st[4][kDecTile][2 + 64 * CH];
   const int split = blockIdx.x, b = blockIdx.z;
@@ -760,7 +788,7 @@ __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
   if (slot == reserved_slot) {
     for (int i = tid; i < nr * Dv; i += 128) {
       const int r = i / Dv, d = i - r * Dv;
-      if (splits == 1) out[((int64_t)b * H + h0 + r) * Dv + d] = from_f<T>(0.f);
+      if (splits == 1) out[(int64_t)b * o_stride + (int64_t)(h0 + r) * Dv + d] = from_f<T>(0.f);
     }
     if (splits > 1 && tid < nr) {
       float* p = part + (((int64_t)b * H + h0 + tid) * splits + split) * rec;
@@ -770,9 +798,9 @@ __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
     return;
   }
   const int pi = positions[b];
-  const int lo = first_key(pi, chunk, db);
-  const int n = pi - lo + 1, per = (n + splits - 1) / splits;
-  const int k_begin = lo + split * per, k_end = min(pi + 1, k_begin + per);
+  const KeyList keys(first_key(pi, chunk, db), pi, db);
+  const int per = (keys.count + splits - 1) / splits;
+  const int k_begin = split * per, k_end = min(keys.count, k_begin + per);   // entries of the list
   for (int i = tid; i < kDecTile * D; i += 128) {
     const int r = i / D, d = i - r * D;
     qs[r][d] = r < nr ? to_f<T>(q[((int64_t)b * H + h0 + r) * D + d]) * (scale * kLog2e) : 0.f;
@@ -820,7 +848,7 @@ __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
   const int n_mine = k_end > k_begin + gid ? (k_end - k_begin - gid + 15) / 16 : 0;
   auto issue = [&](int t) {
     if (t < n_mine) {
-      const int64_t row = cache_row(c, slot, g, k_begin + gid + 16 * t);
+      const int64_t row = cache_row(c, slot, g, keys.pos(k_begin + gid + 16 * t));
       const int stage = t % kStages;
 #pragma unroll
       for (int i = 0; i < CH; ++i) {
@@ -855,7 +883,7 @@ __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
     issue(t + kStages - 1);          // refills the entry the previous pass has finished reading
     cp_async_wait<kStages - 1>();    // everything but the newest kStages - 1 groups has landed: key t is here
     const int stage = t % kStages;
-    const int j = k_begin + gid + 16 * t;
+    const int j = keys.pos(k_begin + gid + 16 * t);
     float s[kDecTile];
 #pragma unroll
     for (int r = 0; r < kDecTile; ++r) s[r] = 0.f;
@@ -962,7 +990,7 @@ __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
       a += st[w][r][2 + d] * f;
     }
     if (splits == 1) {
-      out[((int64_t)b * H + h0 + r) * Dv + d] = from_f<T>(ll > 0.f ? a / ll : 0.f);
+      out[(int64_t)b * o_stride + (int64_t)(h0 + r) * Dv + d] = from_f<T>(ll > 0.f ? a / ll : 0.f);
     } else {
       float* pr = part + (((int64_t)b * H + h0 + r) * splits + split) * rec;
       if (d == 0) { pr[0] = mm; pr[1] = ll; }
@@ -974,7 +1002,8 @@ __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
 template <typename T>
 __global__ void __launch_bounds__(128) bias_attn_decode_merge_kernel(const float* __restrict__ part, float sink,
                                                                      const float* __restrict__ sink_logits, int H,
-                                                                     T* __restrict__ out, int Dv, int splits) {
+                                                                     T* __restrict__ out, int64_t o_stride, int Dv,
+                                                                     int splits) {
   const int64_t bh = blockIdx.x;
   const int rec = 2 + Dv;
   const float* p = part + bh * splits * rec;
@@ -989,35 +1018,35 @@ __global__ void __launch_bounds__(128) bias_attn_decode_merge_kernel(const float
     float a = 0.f;
     for (int s = 0; s < splits; ++s)
       if (p[s * rec] != -INFINITY) a += p[s * rec + 2 + d] * ex2(p[s * rec] - mm);
-    out[bh * Dv + d] = from_f<T>(a * inv);
+    out[bh / H * o_stride + bh % H * Dv + d] = from_f<T>(a * inv);
   }
 }
 
 template <typename T, int CH>
 int launch_decode_split_ch(const void* q, const PagedKV& c, const int32_t* positions, const int32_t* bm,
-                           const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out, float* part, dim3 grid,
-                           int H, int G, int D, int Dv, int splits, int reserved_slot, cudaStream_t st) {
+                           const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out, int64_t o_stride,
+                           float* part, dim3 grid, int H, int G, int D, int Dv, int splits, int reserved_slot, cudaStream_t st) {
   // the ring: stages x (K | V) x CH chunks x 16-byte pieces per chunk x 128 threads x 16 bytes
   const size_t ring = (size_t)(CH <= 2 ? 4 : 2) * 2 * CH * (8 / (16 / sizeof(T))) * 128 * 16;
   static std::atomic<uint64_t> mask{0};
   auto kern = bias_attn_decode_split_kernel<T, CH>;
   CVLLM_CHECK_CUDA(ensure_max_dyn_smem(reinterpret_cast<const void*>(kern), (int)ring, mask));
   kern<<<grid, 128, ring, st>>>(static_cast<const T*>(q), c, positions, bm, slopes, chunk, db, sink, sink_logits, scale,
-                                static_cast<T*>(out), part, H, G, D, Dv, splits, reserved_slot);
+                                static_cast<T*>(out), o_stride, part, H, G, D, Dv, splits, reserved_slot);
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }
 
 template <typename T>
 int launch_decode_split(const void* q, const PagedKV& c, const int32_t* positions, const int32_t* bm,
-                        const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out, float* part, int B, int H,
-                        int G, int D, int Dv, int splits, int reserved_slot, cudaStream_t st) {
+                        const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out, int64_t o_stride,
+                        float* part, int B, int H, int G, int D, int Dv, int splits, int reserved_slot, cudaStream_t st) {
   const int R = H / G, tiles = cdiv(R, kDecTile);
   dim3 grid(splits, G * tiles, B);
   const int ch = cdiv(D > Dv ? D : Dv, 64);
   int rc;
 #define CVLLM_GO(CH) \
-  rc = launch_decode_split_ch<T, CH>(q, c, positions, bm, slopes, chunk, db, sink, sink_logits, scale, out, part, grid, H, G, D, Dv, \
+  rc = launch_decode_split_ch<T, CH>(q, c, positions, bm, slopes, chunk, db, sink, sink_logits, scale, out, o_stride, part, grid, H, G, D, Dv, \
                                      splits, reserved_slot, st)
   if (ch == 1) CVLLM_GO(1);
   else if (ch == 2) CVLLM_GO(2);
@@ -1026,7 +1055,7 @@ int launch_decode_split(const void* q, const PagedKV& c, const int32_t* position
 #undef CVLLM_GO
   if (rc != CVLLM_OK) return rc;
   if (splits > 1) {
-    bias_attn_decode_merge_kernel<T><<<B * H, 128, 0, st>>>(part, sink, sink_logits, H, static_cast<T*>(out), Dv, splits);
+    bias_attn_decode_merge_kernel<T><<<B * H, 128, 0, st>>>(part, sink, sink_logits, H, static_cast<T*>(out), o_stride, Dv, splits);
     CVLLM_CHECK_LAUNCH();
   }
   return CVLLM_OK;
@@ -1039,24 +1068,24 @@ size_t varlen_smem(int BN, int D, int Dv) {
 template <typename T, int BN, int DVC>
 int launch_varlen(const void* q, const PagedKV& c, const int32_t* cu_q, const int32_t* seq_start,
                   const int32_t* batch_mapping, const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out,
-                  int B, int max_new, int H, int G, int D, int Dv, cudaStream_t st) {
+                  int64_t o_stride, int B, int max_new, int H, int G, int D, int Dv, cudaStream_t st) {
   static std::atomic<uint64_t> mask{0};
   const size_t smem = varlen_smem(BN, D, Dv);
   auto kern = bias_attn_varlen_kernel<T, BN, DVC>;
   CVLLM_CHECK_CUDA(ensure_max_dyn_smem(reinterpret_cast<const void*>(kern), 226 * 1024, mask));
   dim3 grid(cdiv(max_new, BM), B, H);
   kern<<<grid, 256, smem, st>>>(static_cast<const T*>(q), c, cu_q, seq_start, batch_mapping, slopes, chunk, db, sink, sink_logits,
-                                scale, static_cast<T*>(out), H, G, D, Dv);
+                                scale, static_cast<T*>(out), o_stride, H, G, D, Dv);
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }
 
 template <typename T, int BN>
 int dispatch_dvc(int dvc, const void* q, const PagedKV& c, const int32_t* cu_q, const int32_t* seq_start,
-                 const int32_t* bm, const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out, int B,
-                 int max_new, int H, int G, int D, int Dv, cudaStream_t st) {
+                 const int32_t* bm, const float* slopes, int chunk, DistBias db, float sink, const float* __restrict__ sink_logits, float scale, void* out,
+                 int64_t o_stride, int B, int max_new, int H, int G, int D, int Dv, cudaStream_t st) {
 #define CVLLM_GO(N) \
-  return launch_varlen<T, BN, N>(q, c, cu_q, seq_start, bm, slopes, chunk, db, sink, sink_logits, scale, out, B, max_new, H, G, D, Dv, st)
+  return launch_varlen<T, BN, N>(q, c, cu_q, seq_start, bm, slopes, chunk, db, sink, sink_logits, scale, out, o_stride, B, max_new, H, G, D, Dv, st)
   if (dvc <= 4) CVLLM_GO(4);
   if (dvc <= 6) CVLLM_GO(6);
   if (dvc <= 8) CVLLM_GO(8);
@@ -1075,8 +1104,8 @@ using namespace cvllm;
 int cvllm_launch_prefill_bias(const void* q, const void* k_cache, const void* v_cache, int64_t cache_rows, void* out,
                               const int32_t* seq_start, const float* slopes, const int32_t* page_table,
                               const int32_t* batch_mapping, const int32_t* cu_seqlens_q, int B, int N, int HQ, int HKV,
-                              int PS, int NLP, int max_seqlen_q, float scale, int chunk, int sink, const float* sink_logits,
-                              cudaStream_t st);
+                              int PS, int NLP, int max_seqlen_q, float scale, int chunk, int window, int keep, int sink,
+                              const float* sink_logits, int64_t o_stride, cudaStream_t st);
 
 static int check_dtype(int dtype) { return dtype == CVLLM_BF16 || dtype == CVLLM_F32; }
 
@@ -1160,8 +1189,8 @@ extern "C" int cvllm_bias_attn_varlen(const void* q, const void* k_cache, const 
                                       int total_tokens, int64_t cache_rows, int pages_per_head, int64_t v_stride,
                                       int dtype, cvllm_stream_t stream) {
   return cvllm_bias_attn_varlen_dist(q, k_cache, v_cache, page_table, table_stride_slot, table_stride_head, page_size,
-                                     cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, 0, nullptr, 0, sink,
-                                     sink_logits, scale, out, B, max_new, H, G, D, Dv, total_tokens, cache_rows,
+                                     cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, 0, 0, nullptr, 0, sink,
+                                     sink_logits, scale, out, 0, B, max_new, H, G, D, Dv, total_tokens, cache_rows,
                                      pages_per_head, v_stride, dtype, stream);
 }
 
@@ -1169,14 +1198,15 @@ extern "C" int cvllm_bias_attn_varlen_dist(const void* q, const void* k_cache, c
                                            const int32_t* page_table, int64_t table_stride_slot,
                                            int64_t table_stride_head, int page_size, const int32_t* cu_seqlens_q,
                                            const int32_t* seq_start, const int32_t* batch_mapping, const float* slopes,
-                                           int chunk, int window, const float* dist_bias, int dist_rows, int sink,
-                                           const float* sink_logits, float scale, void* out, int B, int max_new, int H,
-                                           int G, int D, int Dv, int total_tokens, int64_t cache_rows,
+                                           int chunk, int window, int keep_first, const float* dist_bias, int dist_rows,
+                                           int sink, const float* sink_logits, float scale, void* out,
+                                           int64_t out_stride, int B, int max_new, int H, int G, int D, int Dv, int total_tokens, int64_t cache_rows,
                                            int pages_per_head, int64_t v_stride, int dtype, cvllm_stream_t stream) {
   CVLLM_CHECK_ARG(B >= 0 && max_new >= 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && Dv > 0 && chunk >= 0);
-  CVLLM_CHECK_ARG(window >= 0 && (dist_bias == nullptr || dist_rows > 0));
-  const DistBias db{dist_bias, dist_rows, window};
-  const bool plain_bias = window == 0 && dist_bias == nullptr;   // what the tcgen05 pipeline serves
+  CVLLM_CHECK_ARG(window >= 0 && keep_first >= 0 && (dist_bias == nullptr || dist_rows > 0));
+  const DistBias db{dist_bias, dist_rows, window, keep_first};
+  CVLLM_CHECK_ARG(out_stride == 0 || out_stride >= (int64_t)H * Dv);
+  if (out_stride == 0) out_stride = (int64_t)H * Dv;
   if (B == 0 || max_new == 0) return CVLLM_OK;
   CVLLM_CHECK_ARG(q && k_cache && v_cache && page_table && cu_seqlens_q && seq_start && batch_mapping && out &&
                   check_dtype(dtype) && page_size > 0);
@@ -1190,32 +1220,35 @@ extern "C" int cvllm_bias_attn_varlen_dist(const void* q, const void* k_cache, c
   const float fs = sink ? 1.f : 0.f;
   const size_t cap = 226 * 1024;  // + the static row-index array
   int bn = 64;
-  while (bn > 32 && varlen_smem(bn, D, Dv) > cap) bn >>= 1;
+  while (bn > 16 && varlen_smem(bn, D, Dv) > cap) bn >>= 1;
   CVLLM_CHECK_SUPPORTED(varlen_smem(bn, D, Dv) <= cap);
 #define CVLLM_GO(T, BN) \
-  return dispatch_dvc<T, BN>(dvc, q, c, cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out, B, \
-                             max_new, H, G, D, Dv, st)
+  return dispatch_dvc<T, BN>(dvc, q, c, cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out, \
+                             out_stride, B, max_new, H, G, D, Dv, st)
   const int path = test_options().bias_attn_fma.load();   // 0 product, 1 fp32 FMA kernel, 2 no tcgen05 kernel
   if (dtype == CVLLM_BF16 && D == 128 && Dv == 128 && v_stride == Dv && page_size % 128 == 0 && (H / G) % 2 == 0 &&
-      path == 0 && plain_bias &&
+      path == 0 && dist_bias == nullptr && out_stride % 8 == 0 &&
       table_stride_head == pages_per_head && table_stride_slot == (int64_t)G * pages_per_head && cache_rows > 0)
     return cvllm_launch_prefill_bias(q, k_cache, v_cache, cache_rows, out, seq_start, slopes, page_table,
                                      batch_mapping, cu_seqlens_q, B, total_tokens, H, G, page_size, pages_per_head,
-                                     max_new, scale, chunk, sink, sink_logits, st);
+                                     max_new, scale, chunk, window, keep_first, sink, sink_logits, out_stride, st);
   if (dtype == CVLLM_BF16 && D % 16 == 0 && Dv % 8 == 0 && D <= 128 && Dv <= 128 && path != 1 &&
-      v_stride % vec == 0 && aligned16(k_cache) && aligned16(v_cache)) {
+      v_stride % vec == 0 && aligned16(k_cache) && aligned16(v_cache) && out_stride % 2 == 0 &&
+      reinterpret_cast<uintptr_t>(out) % 4 == 0) {
     if (D <= 64 && Dv <= 64)
-      return launch_varlen_mma<64>(q, c, cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out, B,
-                                   max_new, H, G, D, Dv, st);
-    return launch_varlen_mma<128>(q, c, cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out, B,
-                                  max_new, H, G, D, Dv, st);
+      return launch_varlen_mma<64>(q, c, cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out,
+                                   out_stride, B, max_new, H, G, D, Dv, st);
+    return launch_varlen_mma<128>(q, c, cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out,
+                                  out_stride, B, max_new, H, G, D, Dv, st);
   }
   if (dtype == CVLLM_BF16) {
     if (bn == 64) CVLLM_GO(__nv_bfloat16, 64);
-    CVLLM_GO(__nv_bfloat16, 32);
+    if (bn == 32) CVLLM_GO(__nv_bfloat16, 32);
+    CVLLM_GO(__nv_bfloat16, 16);
   }
   if (bn == 64) CVLLM_GO(float, 64);
-  CVLLM_GO(float, 32);
+  if (bn == 32) CVLLM_GO(float, 32);
+  CVLLM_GO(float, 16);
 #undef CVLLM_GO
 }
 
@@ -1226,8 +1259,8 @@ extern "C" int cvllm_bias_attn_decode(const void* q, const void* k_cache, const 
                                       void* out, int B, int H, int G, int D, int Dv, int reserved_slot, int splits, float* workspace,
                                       size_t workspace_bytes, int64_t v_stride, int dtype, cvllm_stream_t stream) {
   return cvllm_bias_attn_decode_dist(q, k_cache, v_cache, page_table, table_stride_slot, table_stride_head, page_size,
-                                     positions, batch_mapping, slopes, chunk, 0, nullptr, 0, sink, sink_logits, scale,
-                                     out, B, H, G, D, Dv, reserved_slot, splits, workspace, workspace_bytes, v_stride,
+                                     positions, batch_mapping, slopes, chunk, 0, 0, nullptr, 0, sink, sink_logits, scale,
+                                     out, 0, B, H, G, D, Dv, reserved_slot, splits, workspace, workspace_bytes, v_stride,
                                      dtype, stream);
 }
 
@@ -1235,13 +1268,16 @@ extern "C" int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, c
                                            const int32_t* page_table, int64_t table_stride_slot,
                                            int64_t table_stride_head, int page_size, const int32_t* positions,
                                            const int32_t* batch_mapping, const float* slopes, int chunk, int window,
-                                           const float* dist_bias, int dist_rows, int sink, const float* sink_logits,
-                                           float scale, void* out, int B, int H, int G, int D, int Dv,
+                                           int keep_first, const float* dist_bias, int dist_rows, int sink,
+                                           const float* sink_logits, float scale, void* out, int64_t out_stride, int B,
+                                           int H, int G, int D, int Dv,
                                            int reserved_slot, int splits, float* workspace, size_t workspace_bytes,
                                            int64_t v_stride, int dtype, cvllm_stream_t stream) {
   CVLLM_CHECK_ARG(B >= 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && Dv > 0 && chunk >= 0 && splits >= 1);
-  CVLLM_CHECK_ARG(window >= 0 && (dist_bias == nullptr || dist_rows > 0));
-  const DistBias db{dist_bias, dist_rows, window};
+  CVLLM_CHECK_ARG(window >= 0 && keep_first >= 0 && (dist_bias == nullptr || dist_rows > 0));
+  const DistBias db{dist_bias, dist_rows, window, keep_first};
+  CVLLM_CHECK_ARG(out_stride == 0 || out_stride >= (int64_t)H * Dv);
+  if (out_stride == 0) out_stride = (int64_t)H * Dv;
   if (B == 0) return CVLLM_OK;
   CVLLM_CHECK_ARG(q && k_cache && v_cache && page_table && positions && batch_mapping && out && check_dtype(dtype) &&
                   page_size > 0);
@@ -1262,8 +1298,8 @@ extern "C" int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, c
     const float fs = sink ? 1.f : 0.f;
     if (dtype == CVLLM_BF16)
       return launch_decode_split<__nv_bfloat16>(q, c, positions, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out,
-                                                workspace, B, H, G, D, Dv, splits, reserved_slot, st);
-    return launch_decode_split<float>(q, c, positions, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out, workspace, B, H,
+                                                out_stride, workspace, B, H, G, D, Dv, splits, reserved_slot, st);
+    return launch_decode_split<float>(q, c, positions, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out, out_stride, workspace, B, H,
                                       G, D, Dv, splits, reserved_slot, st);
   }
   const size_t smem = sizeof(float) * ((size_t)D + (size_t)kDecWarps * (2 + Dv));
@@ -1272,11 +1308,11 @@ extern "C" int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, c
   if (dtype == CVLLM_BF16)
     bias_attn_decode_kernel<__nv_bfloat16><<<grid, kDecWarps * 32, smem, st>>>(
         static_cast<const __nv_bfloat16*>(q), c, positions, batch_mapping, slopes, chunk, db, sink ? 1.f : 0.f, sink_logits, scale,
-        static_cast<__nv_bfloat16*>(out), H, G, D, Dv, reserved_slot);
+        static_cast<__nv_bfloat16*>(out), out_stride, H, G, D, Dv, reserved_slot);
   else
     bias_attn_decode_kernel<float><<<grid, kDecWarps * 32, smem, st>>>(
         static_cast<const float*>(q), c, positions, batch_mapping, slopes, chunk, db, sink ? 1.f : 0.f, sink_logits, scale,
-        static_cast<float*>(out), H, G, D, Dv, reserved_slot);
+        static_cast<float*>(out), out_stride, H, G, D, Dv, reserved_slot);
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }

@@ -86,7 +86,7 @@ __global__ void __launch_bounds__(kThreads) sandwich_norm_kernel(
 // One CTA per row of a 32-bit residual stream:
 //   resid += a + b + c     (a, b [rows, width] of type TY, c fp32; each may be NULL)
 //   out = norm(resid)      (out may be NULL: the sum alone)
-// KIND 0: resid / sqrt(mean(resid^2) + eps) * w;   KIND 1, layer norm: (resid - mean) / sqrt(var + eps) * w + bias with
+// KIND 0: resid / sqrt(mean(resid^2) + eps) * w;   KIND 2: the same with ONE gain w[0] for all coordinates;   KIND 1, layer norm: (resid - mean) / sqrt(var + eps) * w + bias with
 // var = the mean of the squared deviations (second pass over the row held in shared memory).  Sum, statistics and the
 // stream are fp32 whatever the activations' type.
 template <typename TY, typename TO, int KIND>
@@ -112,9 +112,10 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(
   if (out == nullptr) return;
   TO* o = out + r * o_stride;
   s1 = block_sum(s1, red);
-  if constexpr (KIND == 0) {
+  if constexpr (KIND != 1) {
     const float inv = 1.0f / sqrtf(s1 / (float)width + eps);
-    for (int i = threadIdx.x; i < width; i += kThreads) o[i] = from_f<TO>(row[i] * inv * w[i]);
+    const float w0 = w[0];
+    for (int i = threadIdx.x; i < width; i += kThreads) o[i] = from_f<TO>(row[i] * inv * (KIND == 2 ? w0 : w[i]));
   } else {
     const float mean = s1 / (float)width;
     float s2 = 0.f;
@@ -127,6 +128,40 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(
     for (int i = threadIdx.x; i < width; i += kThreads)
       o[i] = from_f<TO>((row[i] - mean) * inv * w[i] + (bias ? bias[i] : 0.f));
   }
+}
+
+// Token embedding, normed, as the start of a 32-bit residual stream, one CTA per token:
+//   resid[t, :] = rms(embed[id_t, :]) * w_embed;   out[t, :] = rms(resid[t, :]) * w_next   (out NULL: the stream alone)
+// with rms(x) = x / sqrt(mean(x^2) + eps).  one_gain: both weights are a single number.
+template <typename T, typename TO>
+__global__ void __launch_bounds__(kThreads) embed_norm_kernel(
+    const int64_t* __restrict__ ids, const T* __restrict__ embed, const float* __restrict__ w_embed,
+    const float* __restrict__ w_next, int one_gain, float* __restrict__ resid, int64_t r_stride, TO* __restrict__ out,
+    int64_t o_stride, int width, float eps) {
+  extern __shared__ float row[];
+  __shared__ float red[kThreads / 32];
+  const int64_t t = blockIdx.x;
+  const T* e = embed + ids[t] * width;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < width; i += kThreads) {
+    const float v = to_f<T>(e[i]);
+    row[i] = v;
+    ss += v * v;
+  }
+  ss = block_sum(ss, red);
+  float inv = 1.0f / sqrtf(ss / (float)width + eps);
+  ss = 0.f;
+  for (int i = threadIdx.x; i < width; i += kThreads) {   // every thread reads back what it wrote itself
+    const float v = row[i] * inv * w_embed[one_gain ? 0 : i];
+    resid[t * r_stride + i] = v;
+    row[i] = v;
+    ss += v * v;
+  }
+  if (out == nullptr) return;
+  ss = block_sum(ss, red);
+  inv = 1.0f / sqrtf(ss / (float)width + eps);
+  for (int i = threadIdx.x; i < width; i += kThreads)
+    out[t * o_stride + i] = from_f<TO>(row[i] * inv * w_next[one_gain ? 0 : i]);
 }
 
 // Token embedding plus a hashed embedding of the (previous token, token) pair, one CTA per token:
@@ -545,7 +580,7 @@ extern "C" int cvllm_residual_norm(const void* a, int64_t a_stride, const void* 
                                    const float* bias, void* out, int64_t o_stride, int out_dtype, int rows, int width,
                                    float eps, int kind, cvllm_stream_t stream) {
   drop_stale_error();
-  CVLLM_CHECK_ARG(rows >= 0 && width > 0 && resid && (kind == 0 || kind == 1));
+  CVLLM_CHECK_ARG(rows >= 0 && width > 0 && resid && kind >= 0 && kind <= 2);
   if (rows == 0) return CVLLM_OK;
   CVLLM_CHECK_ARG((a == nullptr && b == nullptr) || ab_dtype == CVLLM_BF16 || ab_dtype == CVLLM_F32);
   CVLLM_CHECK_ARG(out == nullptr || (w != nullptr && (out_dtype == CVLLM_BF16 || out_dtype == CVLLM_F32)));
@@ -558,13 +593,42 @@ extern "C" int cvllm_residual_norm(const void* a, int64_t a_stride, const void* 
       static_cast<const TY*>(a), a_stride, static_cast<const TY*>(b), b_stride, c, c_stride, resid, r_stride, w,    \
       bias, static_cast<TO*>(out), o_stride, width, eps)
 #define CVLLM_RESNORM_K(TY, TO) \
-  do { if (kind == 0) CVLLM_RESNORM(TY, TO, 0); else CVLLM_RESNORM(TY, TO, 1); } while (0)
+  do {                                        \
+    if (kind == 0) CVLLM_RESNORM(TY, TO, 0);  \
+    else if (kind == 1) CVLLM_RESNORM(TY, TO, 1); \
+    else CVLLM_RESNORM(TY, TO, 2);            \
+  } while (0)
   if (yb && ob) CVLLM_RESNORM_K(__nv_bfloat16, __nv_bfloat16);
   else if (yb) CVLLM_RESNORM_K(__nv_bfloat16, float);
   else if (ob) CVLLM_RESNORM_K(float, __nv_bfloat16);
   else CVLLM_RESNORM_K(float, float);
 #undef CVLLM_RESNORM_K
 #undef CVLLM_RESNORM
+  CVLLM_CHECK_LAUNCH();
+  return CVLLM_OK;
+}
+
+extern "C" int cvllm_embed_norm(const int64_t* ids, const void* embed, int dtype, const float* w_embed,
+                                const float* w_next, int one_gain, float* resid, int64_t r_stride, void* out,
+                                int64_t o_stride, int out_dtype, int T, int width, float eps, cvllm_stream_t stream) {
+  drop_stale_error();
+  CVLLM_CHECK_ARG(T >= 0 && width > 0);
+  if (T == 0) return CVLLM_OK;
+  CVLLM_CHECK_ARG(ids && embed && w_embed && resid && (dtype == CVLLM_BF16 || dtype == CVLLM_F32));
+  CVLLM_CHECK_ARG(out == nullptr || (w_next != nullptr && (out_dtype == CVLLM_BF16 || out_dtype == CVLLM_F32)));
+  CVLLM_CHECK_SUPPORTED(width <= 12288);
+  auto st = static_cast<cudaStream_t>(stream);
+  const size_t smem = (size_t)width * sizeof(float);
+#define CVLLM_EMBNORM(T_, TO)                                                                                   \
+  embed_norm_kernel<T_, TO><<<T, kThreads, smem, st>>>(ids, static_cast<const T_*>(embed), w_embed, w_next, one_gain, \
+                                                       resid, r_stride, static_cast<TO*>(out), o_stride, width, eps)
+  const bool ob = out != nullptr && out_dtype == CVLLM_BF16;
+  if (dtype == CVLLM_BF16) {
+    if (ob) CVLLM_EMBNORM(__nv_bfloat16, __nv_bfloat16); else CVLLM_EMBNORM(__nv_bfloat16, float);
+  } else {
+    if (ob) CVLLM_EMBNORM(float, __nv_bfloat16); else CVLLM_EMBNORM(float, float);
+  }
+#undef CVLLM_EMBNORM
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }

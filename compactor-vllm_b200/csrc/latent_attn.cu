@@ -7,6 +7,9 @@
 //   cvllm_latent_norm_store   RMS norm of the query latent; RMS norm of the kv latent, rotation of the shared key
 //                             part, both written to the token's cache row
 //   cvllm_latent_q_rope       rotation of every head's rotated query part into the attention's query rows
+//   cvllm_latent_prepare      for queries without a latent of their own: the kv latent's norm, the rotation of the
+//                             shared key part and of every head's query part and the cache write in one launch, with
+//                             a choice of pairing and a factor on sine and cosine
 //   cvllm_sigmoid_gate        x * sigmoid(gate), element by element
 // Rotation ("rotate half"): element i of a part of R numbers pairs with element i + R/2; the pair (u, v) at position
 // p becomes (u cos a - v sin a, v cos a + u sin a), a = p * inv_freq[i].  Angles and their sines are computed in
@@ -126,6 +129,107 @@ __global__ void __launch_bounds__(kThreads) latent_q_rope_kernel(
   }
 }
 
+// One CTA per token.  proj row: H query heads of D + R numbers at q_off (the last R of each are rotated into
+// q_full[t, h, off ..]; the first D are left to the change of basis), the kv latent and the shared key part at kv_off.
+// Warp 0 norms the latent and writes the cache row, the other warps rotate the query parts.  neighbours: the pair i is
+// (2i, 2i + 1) instead of (i, i + R / 2).  Sine and cosine are multiplied by amp.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) latent_prepare_kernel(
+    const T* __restrict__ proj, int64_t p_stride, int q_off, int H, int D, int kv_off, int kv_rank, int R,
+    const float* __restrict__ kv_w, float eps, const double* __restrict__ inv_freq, float amp, int neighbours,
+    const int32_t* __restrict__ positions, const int32_t* __restrict__ token_slot, T* __restrict__ q_full,
+    int64_t f_stride, int f_head, int off, T* __restrict__ cache, const int32_t* __restrict__ table,
+    int64_t table_stride_slot, int page_size, int32_t* __restrict__ lens, int reserved_slot) {
+  extern __shared__ float sm[];     // cos[R/2], sin[R/2]
+  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* row = proj + (int64_t)t * p_stride;
+  const int half = R / 2;
+  float* cs = sm;
+  float* sn = sm + half;
+  const int pos = positions[t], slot = token_slot[t];
+  for (int i = threadIdx.x; i < half; i += kThreads) {
+    double sv, cv;
+    sincos((double)pos * inv_freq[i], &sv, &cv);
+    cs[i] = (float)cv * amp;
+    sn[i] = (float)sv * amp;
+  }
+  __syncthreads();
+  const int step = neighbours ? 1 : half;     // distance of a pair's two numbers
+  if (warp == 0) {
+    if (slot == reserved_slot) return;
+    const int lp = pos / page_size;
+    const int page = table[(int64_t)slot * table_stride_slot + lp];
+    T* dst = cache + ((int64_t)page * page_size + (pos - lp * page_size)) * (kv_rank + R);
+    const T* c = row + kv_off;
+    float ss = 0.f;
+    for (int i = lane; i < kv_rank; i += 32) {
+      const float v = to_f<T>(c[i]);
+      ss += v * v;
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)kv_rank + eps);
+    for (int i = lane; i < kv_rank; i += 32) dst[i] = from_f<T>(to_f<T>(c[i]) * inv * kv_w[i]);
+    for (int i = lane; i < half; i += 32) {
+      const int a = neighbours ? 2 * i : i;
+      const float u = to_f<T>(c[kv_rank + a]), v = to_f<T>(c[kv_rank + a + step]);
+      dst[kv_rank + a] = from_f<T>(u * cs[i] - v * sn[i]);
+      dst[kv_rank + a + step] = from_f<T>(v * cs[i] + u * sn[i]);
+    }
+    if (lane == 0 && lens) atomicMax(lens + slot, pos + 1);
+    return;
+  }
+  for (int k = threadIdx.x - 32; k < H * half; k += kThreads - 32) {
+    const int h = k / half, i = k - h * half;
+    const int a = neighbours ? 2 * i : i;
+    const T* src = row + q_off + (int64_t)h * (D + R) + D + a;
+    T* dst = q_full + (int64_t)t * f_stride + (int64_t)h * f_head + off + a;
+    const float u = to_f<T>(src[0]), v = to_f<T>(src[step]);
+    dst[0] = from_f<T>(u * cs[i] - v * sn[i]);
+    dst[step] = from_f<T>(v * cs[i] + u * sn[i]);
+  }
+}
+
+// eight numbers as one 16-byte (32-bit type: two) access
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float* v) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    v[2 * i] = __uint_as_float(w[i] << 16);
+    v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
+__device__ __forceinline__ void load8(const float* p, float* v) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float* v) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack2<true>(v[0], v[1]), pack2<true>(v[2], v[3]), pack2<true>(v[4], v[5]),
+                                            pack2<true>(v[6], v[7]));
+}
+__device__ __forceinline__ void store8(float* p, const float* v) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+
+// width and every stride a multiple of 8, rows 16-byte aligned: a thread takes eight neighbours
+template <typename T>
+__global__ void sigmoid_gate_vec_kernel(const T* __restrict__ x, int64_t x_stride, const T* __restrict__ g,
+                                        int64_t g_stride, T* __restrict__ out, int64_t o_stride, int64_t rows,
+                                        int width8) {
+  const int64_t total = rows * (int64_t)width8;
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = i / width8;
+    const int c = (int)(i - t * width8) * 8;
+    float xv[8], gv[8];
+    load8(x + t * x_stride + c, xv);
+    load8(g + t * g_stride + c, gv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) xv[e] = xv[e] / (1.0f + expf(-gv[e]));
+    store8(out + t * o_stride + c, xv);
+  }
+}
+
 template <typename T>
 __global__ void sigmoid_gate_kernel(const T* __restrict__ x, int64_t x_stride, const T* __restrict__ g,
                                     int64_t g_stride, T* __restrict__ out, int64_t o_stride, int64_t rows, int width) {
@@ -195,16 +299,56 @@ extern "C" int cvllm_latent_q_rope(const void* q, int64_t q_stride, int H, int D
   return CVLLM_OK;
 }
 
+extern "C" int cvllm_latent_prepare(const void* proj, int64_t proj_stride, int q_off, int H, int D, int kv_off,
+                                    int kv_rank, int rot_dim, const float* kv_weight, float eps, const double* inv_freq,
+                                    float amplitude, int neighbours, const int32_t* positions,
+                                    const int32_t* token_slot, void* q_full, int64_t full_stride, int full_head, int off,
+                                    void* cache, const int32_t* page_table, int64_t table_stride_slot, int page_size,
+                                    int32_t* lens, int T, int reserved_slot, int dtype, cvllm_stream_t stream) {
+  CVLLM_CHECK_ARG(T >= 0 && H > 0 && D >= 0 && kv_rank > 0 && rot_dim >= 0 && rot_dim % 2 == 0 && q_off >= 0 &&
+                  kv_off >= 0 && off >= 0 && off + rot_dim <= full_head);
+  if (T == 0) return CVLLM_OK;
+  CVLLM_CHECK_ARG(proj && kv_weight && positions && token_slot && q_full && cache && page_table && page_size > 0 &&
+                  (rot_dim == 0 || inv_freq) && latent_dtype_ok(dtype));
+  auto st = static_cast<cudaStream_t>(stream);
+  const size_t smem = (size_t)rot_dim * sizeof(float);
+  CVLLM_CHECK_SUPPORTED(smem <= 48 * 1024);
+  if (dtype == CVLLM_BF16)
+    latent_prepare_kernel<__nv_bfloat16><<<T, kThreads, smem, st>>>(
+        static_cast<const __nv_bfloat16*>(proj), proj_stride, q_off, H, D, kv_off, kv_rank, rot_dim, kv_weight, eps,
+        inv_freq, amplitude, neighbours, positions, token_slot, static_cast<__nv_bfloat16*>(q_full), full_stride,
+        full_head, off, static_cast<__nv_bfloat16*>(cache), page_table, table_stride_slot, page_size, lens,
+        reserved_slot);
+  else
+    latent_prepare_kernel<float><<<T, kThreads, smem, st>>>(
+        static_cast<const float*>(proj), proj_stride, q_off, H, D, kv_off, kv_rank, rot_dim, kv_weight, eps, inv_freq,
+        amplitude, neighbours, positions, token_slot, static_cast<float*>(q_full), full_stride, full_head, off,
+        static_cast<float*>(cache), page_table, table_stride_slot, page_size, lens, reserved_slot);
+  CVLLM_CHECK_LAUNCH();
+  return CVLLM_OK;
+}
+
 extern "C" int cvllm_sigmoid_gate(const void* x, int64_t x_stride, const void* gate, int64_t g_stride, void* out,
                                   int64_t o_stride, int64_t rows, int width, int dtype, cvllm_stream_t stream) {
   CVLLM_CHECK_ARG(rows >= 0 && width > 0);
   if (rows == 0) return CVLLM_OK;
   CVLLM_CHECK_ARG(x && gate && out && latent_dtype_ok(dtype));
   auto st = static_cast<cudaStream_t>(stream);
-  const int64_t total = rows * (int64_t)width;
+  const bool vec = width % 8 == 0 && x_stride % 8 == 0 && g_stride % 8 == 0 && o_stride % 8 == 0 && aligned16(x) &&
+                   aligned16(gate) && aligned16(out);
+  const int64_t total = rows * (int64_t)(vec ? width / 8 : width);
   const int64_t want = (total + 255) / 256, cap = (int64_t)sm_count() * 16;
   const int grid = (int)(want < cap ? want : cap);
-  if (dtype == CVLLM_BF16)
+  if (vec) {
+    if (dtype == CVLLM_BF16)
+      sigmoid_gate_vec_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(
+          static_cast<const __nv_bfloat16*>(x), x_stride, static_cast<const __nv_bfloat16*>(gate), g_stride,
+          static_cast<__nv_bfloat16*>(out), o_stride, rows, width / 8);
+    else
+      sigmoid_gate_vec_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(x), x_stride,
+                                                           static_cast<const float*>(gate), g_stride,
+                                                           static_cast<float*>(out), o_stride, rows, width / 8);
+  } else if (dtype == CVLLM_BF16)
     sigmoid_gate_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(
         static_cast<const __nv_bfloat16*>(x), x_stride, static_cast<const __nv_bfloat16*>(gate), g_stride,
         static_cast<__nv_bfloat16*>(out), o_stride, rows, width);

@@ -4,9 +4,10 @@
 // issuer), same ring of five 32 KB slots, same TMEM layout and hand-offs; what differs:
 //   * every key - the step's own tokens included - is already in the paged cache, so all K / V tiles are cache tiles
 //     [128 j, 128 j + 127] of the sequence and the causal mask is positional: key position <= query position;
-//   * tiles before the chunk of the query tile's first row are never loaded (the tile loop starts at j_begin);
+//   * tiles before the chunk (or the sliding window) of the query tile's first row are never loaded: the tile list is
+//     the tiles that hold kept first tokens, if any, then the tiles from j_begin on;
 //   * the softmax adds slope * (key position - query position) in log2 units to the scaled logits, masks keys outside
-//     the row's chunk, and starts from (max 0, sum 1) when there is a sink.
+//     the row's chunk or window (the kept first tokens stay visible), and starts from (max 0, sum 1) when there is a sink.
 #include <stdlib.h>
 
 #include "common.cuh"
@@ -35,6 +36,8 @@ struct PrefillBiasParams {
   float scale_log2;
   float rescale_threshold;
   int chunk;                  // 0 = no chunking
+  int window;                 // keys at distances 0 .. window - 1 (0 = no limit)
+  int keep;                   // the sequence's first positions that stay visible whatever window and chunk say
   float sink;                 // 1 = a sink in the denominator, 0 = none
   const float* sink_logits;   // [HQ] the sink's score per head, or NULL (score 0)
 };
@@ -116,8 +119,17 @@ prefill_attn_bias_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
   const int q0 = qt * kBM;
   const int p0 = p.seq_start[b] + q0;                      // position of the tile's first query
   const int p_last = p0 + min(kBM, La - q0) - 1;           // ... and of its last valid one
-  const int j_begin = (p.chunk > 0 ? (p0 / p.chunk) * p.chunk : 0) / kBN;
-  const int n_tiles = p_last / kBN - j_begin + 1;          // key tiles j_begin .. p_last / 128
+  auto first_key = [&](int pi) {                           // first position a query at pi sees through chunk and window
+    int lo = p.chunk > 0 ? (pi / p.chunk) * p.chunk : 0;
+    if (p.window > 0) lo = max(lo, pi - p.window + 1);
+    return lo;
+  };
+  const int lo0 = first_key(p0);
+  const int j_begin = lo0 / kBN;
+  const int n_kept = min((min(p.keep, lo0) + kBN - 1) / kBN, j_begin);   // tiles of kept first tokens before j_begin
+  const int n_tiles = n_kept + p_last / kBN - j_begin + 1;               // then the tiles j_begin .. p_last / 128
+  const int j_skip = j_begin - n_kept;
+  auto tile_base = [&](int j) { return (j < n_kept ? j : j + j_skip) * kBN; };   // first position of the list's tile j
   const int last_valid = p_last + 1 - (p_last / kBN) * kBN;  // keys of the last tile at or before p_last
 
   // ---------------- setup ----------------
@@ -166,7 +178,7 @@ prefill_attn_bias_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
         const bool is_v = n & 1;
         const int slot = n % kSlots;
         const uint32_t ph = (n / kSlots) & 1;
-        const int t0 = (j_begin + j) * kBN;
+        const int t0 = tile_base(j);
         const int pg = t0 / p.PS;
         const int row = pt[pg] * p.PS + (t0 - pg * p.PS);
         mbar_wait(&sm.empty[slot], ph ^ 1);
@@ -295,8 +307,8 @@ prefill_attn_bias_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
     float m_ref = p.sink > 0.f ? (p.sink_logits ? p.sink_logits[hq0 + t] * 1.4426950408889634f : 0.f) : -INFINITY;
     float l = p.sink;
     const int pi = p0 + row;                                   // this thread's query position
-    const int lo_i = p.chunk > 0 ? (pi / p.chunk) * p.chunk : 0;
-    const int lo_max = p.chunk > 0 ? (p_last / p.chunk) * p.chunk : 0;
+    const int lo_i = first_key(pi);
+    const int lo_max = first_key(p_last);
     const float slope2 = p.slopes ? p.slopes[hq0 + t] * 1.4426950408889634f : 0.f;
 
     for (int j = 0; j < n_tiles; ++j) {
@@ -321,7 +333,7 @@ prefill_attn_bias_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
       tc_wait_ld();
 
       // ---- logits in log2 units with the distance bias: s_c * scale + slope2 * (pj - pi), pj = base + c ----
-      const int base = (j_begin + j) * kBN;
+      const int base = tile_base(j);
       {
         const float2 sc2 = make_float2(p.scale_log2, p.scale_log2), sl2 = make_float2(slope2, slope2);
         const float off = slope2 * (float)(base - pi);
@@ -334,12 +346,13 @@ prefill_attn_bias_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
           s[c + 1] = v.y;
         }
       }
-      // ---- masks (boundary tiles only): keys after the query, keys before the row's chunk ----
+      // ---- masks (boundary tiles only): keys after the query, keys before the row's chunk or window ----
       if (base + kBN - 1 > p0 || base < lo_max) {
-        const int c_hi = pi - base, c_lo = lo_i - base;   // visible columns: c_lo <= c <= c_hi
+        const int c_hi = pi - base, c_lo = lo_i - base;   // visible columns: c_lo <= c <= c_hi, and kept ones
+        const int c_keep = p.keep - base;
 #pragma unroll
         for (int c = 0; c < kBN; ++c)
-          if (c > c_hi || c < c_lo) s[c] = -INFINITY;
+          if (c > c_hi || (c < c_lo && c >= c_keep)) s[c] = -INFINITY;
       }
 
       auto row_max = [&]() -> float {
@@ -351,7 +364,7 @@ prefill_attn_bias_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_
           mx2 = fmaxf(mx2, s[c + 2]);
           mx3 = fmaxf(mx3, s[c + 3]);
         }
-        // a row that sees no key of this tile (it lies in a later chunk) keeps a finite reference
+        // a row that sees no key of this tile (it lies before the row's chunk or window) keeps a finite reference
         return fmaxf(fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)), -1e30f);
       };
       // O *= alpha, l *= alpha, m_ref <- m_to.  O holds PV(0..j-1); PV(j-1) may still be in flight.
@@ -475,8 +488,8 @@ using namespace cvllm;
 int cvllm_launch_prefill_bias(const void* q, const void* k_cache, const void* v_cache, int64_t cache_rows, void* out,
                               const int32_t* seq_start, const float* slopes, const int32_t* page_table,
                               const int32_t* batch_mapping, const int32_t* cu_seqlens_q, int B, int N, int HQ, int HKV,
-                              int PS, int NLP, int max_seqlen_q, float scale, int chunk, int sink, const float* sink_logits,
-                              cudaStream_t st) {
+                              int PS, int NLP, int max_seqlen_q, float scale, int chunk, int window, int keep, int sink,
+                              const float* sink_logits, int64_t o_stride, cudaStream_t st) {
   using namespace pb;
   CVLLM_CHECK_ALIGN(aligned16(q) && aligned16(out) && aligned16(k_cache) && aligned16(v_cache));
   CUtensorMap tm_q, tm_kc, tm_vc;
@@ -498,7 +511,7 @@ int cvllm_launch_prefill_bias(const void* q, const void* k_cache, const void* v_
   p.out = out; p.seq_start = seq_start; p.slopes = slopes; p.page_table = page_table;
   p.batch_mapping = batch_mapping; p.cu_seqlens_q = cu_seqlens_q;
   p.B = B; p.HQ = HQ; p.HKV = HKV; p.G = HQ / HKV; p.PS = PS; p.NLP = NLP;
-  p.o_stride_n = (int64_t)HQ * kHD;
+  p.o_stride_n = o_stride;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.rescale_threshold = 8.0f;
   {
@@ -506,6 +519,8 @@ int cvllm_launch_prefill_bias(const void* q, const void* k_cache, const void* v_
     if (t >= 0.f) p.rescale_threshold = t;
   }
   p.chunk = chunk;
+  p.window = window;
+  p.keep = keep;
   p.sink = sink ? 1.f : 0.f;
   p.sink_logits = sink ? sink_logits : nullptr;
   const size_t smem = sizeof(PrefillBiasSmem) + 1024;

@@ -418,11 +418,18 @@ int cvllm_sandwich_norm(const void* y, int64_t y_stride, int y_dtype, const floa
  *   resid += a + b + c   (a, b [rows, width] of ab_dtype, c fp32 [rows, width]; each may be NULL)
  *   out = norm(resid)    (out may be NULL: the sum alone); kind 0: resid / sqrt(mean(resid^2) + eps) * w;
  *   kind 1, layer norm: (resid - mean) / sqrt(var + eps) * w + bias, var = the mean of the squared deviations
- *   (bias may be NULL).  w, bias fp32.  width <= 12288.  Strides in elements. */
+ *   (bias may be NULL); kind 2: kind 0 with one gain w[0] for all coordinates.  w, bias fp32.  width <= 12288.  Strides in elements. */
 int cvllm_residual_norm(const void* a, int64_t a_stride, const void* b, int64_t b_stride, int ab_dtype,
                         const float* c, int64_t c_stride, float* resid, int64_t r_stride, const float* w,
                         const float* bias, void* out, int64_t o_stride, int out_dtype, int rows, int width, float eps,
                         int kind, cvllm_stream_t stream);
+
+/* The start of a 32-bit residual stream from a normed token embedding: resid[t, :] = rms(embed[ids[t], :]) * w_embed and
+ * (out not NULL) out[t, :] = rms(resid[t, :]) * w_next, rms(x) = x / sqrt(mean(x^2) + eps).  embed [V, width] of `dtype`,
+ * weights fp32 [width], or a single number each when one_gain is set.  width <= 12288. */
+int cvllm_embed_norm(const int64_t* ids, const void* embed, int dtype, const float* w_embed, const float* w_next,
+                     int one_gain, float* resid, int64_t r_stride, void* out, int64_t o_stride, int out_dtype, int T,
+                     int width, float eps, cvllm_stream_t stream);
 
 /* out[t, :] (fp32) = embed[ids[t], :] + pair[row_t, :] with row_t = (prev_t * mul_prev + ids[t] * mul_cur) mod buckets,
  * and row_t = buckets (the table's extra last row) where positions[t] == 0.  prev_t = ids[t - 1] when token t - 1 of
@@ -488,7 +495,8 @@ int cvllm_qknorm_store(const void* qkv, int64_t qkv_stride, const float* q_weigh
 
 /* The same with a rotation in front of the norm: inv_freq [rot_dims / 2] doubles (NULL = none); neighbours
  * (2 i, 2 i + 1) of the first rot_dims numbers of every q and k head turn by positions[t] * inv_freq[i].
- * norm 0: no norm at all; 1: the RMS norm above (weights may be NULL). */
+ * norm is a bit mask: bit 0, the RMS norm above on q and k (weights may be NULL); bit 1, values are stored divided by
+ * their root mean square, x / sqrt(mean(x^2) + eps) over Dv. */
 int cvllm_rope_qknorm_store(const void* qkv, int64_t qkv_stride, const double* inv_freq, int rot_dims, int norm,
                             const float* q_weight, const float* k_weight, float eps, const int32_t* positions,
                             const int32_t* token_slot, void* q_out, void* k_cache, void* v_cache,
@@ -525,21 +533,23 @@ int cvllm_bias_attn_decode(const void* q, const void* k_cache, const void* v_cac
 /* The same two with a sliding window and a learned bias per distance beside the linear bias and the chunk mask:
  * a query sees the keys at distances 0 .. window - 1 (window 0: no limit), and the score of the key at distance n
  * gets dist_bias[min(n, dist_rows - 1), h] (fp32 [dist_rows, H]; NULL = none), unscaled.  The caller makes the
- * table, so any rule from distance to bias (buckets of a smaller learned table) is served.  These shapes run on the
- * mma.sync and fp32 FMA kernels. */
+ * table, so any rule from distance to bias (buckets of a smaller learned table) is served.  keep_first > 0: the
+ * sequence's first keep_first positions stay visible to every later query whatever window and chunk say.  out_stride:
+ * elements between the outputs of neighbouring tokens (0 = H * Dv).  A bias table runs on the mma.sync and fp32 FMA
+ * kernels only; windows and kept tokens on all of them. */
 int cvllm_bias_attn_varlen_dist(const void* q, const void* k_cache, const void* v_cache, const int32_t* page_table,
                                 int64_t table_stride_slot, int64_t table_stride_head, int page_size,
                                 const int32_t* cu_seqlens_q, const int32_t* seq_start, const int32_t* batch_mapping,
-                                const float* slopes, int chunk, int window, const float* dist_bias, int dist_rows,
-                                int sink, const float* sink_logits, float scale, void* out, int B, int max_new, int H,
-                                int G, int D, int Dv, int total_tokens, int64_t cache_rows, int pages_per_head,
+                                const float* slopes, int chunk, int window, int keep_first,
+                                const float* dist_bias, int dist_rows, int sink, const float* sink_logits, float scale,
+                                void* out, int64_t out_stride, int B, int max_new, int H, int G, int D, int Dv, int total_tokens, int64_t cache_rows, int pages_per_head,
                                 int64_t v_stride, int dtype, cvllm_stream_t stream);
 int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, const void* v_cache, const int32_t* page_table,
                                 int64_t table_stride_slot, int64_t table_stride_head, int page_size,
                                 const int32_t* positions, const int32_t* batch_mapping, const float* slopes, int chunk,
-                                int window, const float* dist_bias, int dist_rows, int sink, const float* sink_logits,
-                                float scale, void* out, int B, int H, int G, int D, int Dv, int reserved_slot,
-                                int splits, float* workspace, size_t workspace_bytes, int64_t v_stride, int dtype,
+                                int window, int keep_first, const float* dist_bias, int dist_rows, int sink,
+                                const float* sink_logits, float scale, void* out, int64_t out_stride, int B, int H,
+                                int G, int D, int Dv, int reserved_slot, int splits, float* workspace, size_t workspace_bytes, int64_t v_stride, int dtype,
                                 cvllm_stream_t stream);
 
 /* ------------------------------------------------------------------------
@@ -563,6 +573,18 @@ int cvllm_latent_norm_store(const void* proj, int64_t proj_stride, int q_off, in
 int cvllm_latent_q_rope(const void* q, int64_t q_stride, int H, int D, int rot_dim, const double* inv_freq,
                         const int32_t* positions, void* q_full, int64_t full_stride, int full_head, int off, int T,
                         int dtype, cvllm_stream_t stream);
+
+/* The same steps for queries without a latent of their own, in one launch: proj rows hold H query heads of D + rot_dim
+ * numbers at q_off and the kv latent followed by the shared key part at kv_off.  Writes the cache row as above (norm
+ * weight kv_weight) and q_full[t * full_stride + h * full_head + off + 0 .. rot_dim) = the rotated last rot_dim numbers
+ * of every query head.  neighbours 0: number i pairs with i + rot_dim / 2; 1: 2 i pairs with 2 i + 1.  Sine and cosine
+ * are multiplied by `amplitude`. */
+int cvllm_latent_prepare(const void* proj, int64_t proj_stride, int q_off, int H, int D, int kv_off, int kv_rank,
+                         int rot_dim, const float* kv_weight, float eps, const double* inv_freq, float amplitude,
+                         int neighbours, const int32_t* positions, const int32_t* token_slot, void* q_full,
+                         int64_t full_stride, int full_head, int off, void* cache, const int32_t* page_table,
+                         int64_t table_stride_slot, int page_size, int32_t* lens, int T, int reserved_slot, int dtype,
+                         cvllm_stream_t stream);
 
 /* Gated residual sum fused with the next RMS norm, one launch on a 32-bit residual stream [rows, width]:
  *   resid += sigmoid(gate) * y   (y, gate [rows, width] bfloat16 or float32; both NULL: no sum)
