@@ -111,7 +111,8 @@ _SIGNATURES = {
     "cvllm_bias_attn_varlen_dist": (_i, [_p, _p, _p, _p, _i64, _i64, _i, _p, _p, _p, _p, _i, _i, _i, _p, _i, _i, _p, _f,
                                          _p, _i64, _i, _i, _i, _i, _i, _i, _i, _i64, _i, _i64, _i, _p]),
     "cvllm_bias_attn_decode_dist": (_i, [_p, _p, _p, _p, _i64, _i64, _i, _p, _p, _p, _i, _i, _i, _p, _i, _i, _p, _f, _p,
-                                         _i64, _i, _i, _i, _i, _i, _i, _i, _p, _sz, _i64, _i, _p]),
+                                         _i64, _i, _i, _i, _i, _i, _i64, _i, _i, _p, _sz, _i64, _i, _p]),
+    "cvllm_latent_attn_aborts": (_i, [_p]),
     "cvllm_general_delta": (_i, [_p, _i64, _i, _i, _i, _i, _p, _i64, _p, _f, _p, _i, _i, _p, _i, _f, _p, _p, _p, _p,
                                  _i, _i, _p, _i64, _i, _i, _i, _i, _p]),
     "cvllm_matrix_memory": (_i, [_p, _i64, _i, _i, _i, _i, _i, _f, _f, _p, _p, _p, _i, _i, _p, _i, _f, _p, _p, _p, _p,

@@ -270,10 +270,22 @@ class BiasedChunkAttention(nn.Module):
         if self.window:
             keys = min(keys, self.window)
         keys = min(keys + self.keep_first, max_keys)
+        if self.wide_latent_rows:
+            # the tcgen05 kernel for wide latent rows: a CTA per (128 heads, 256 value columns, split), tiles of 64 keys
+            ctas = max(batch * -(-self.num_heads // 128) * -(-self.v_head_dim // 256), 1)
+            return int(max(1, min(148 // ctas, keys // 128, 64)))
         ctas = max(batch * self.num_kv_heads * -(-(self.num_heads // self.num_kv_heads) // 4), 1)
         one_wave = min(296 // ctas, keys // 128)
         several = min(2048 // ctas, keys // 1024)
         return int(max(1, min(max(one_wave, several), 64)))
+
+    @property
+    def wide_latent_rows(self) -> bool:
+        """Whether csrc/latent_attn_umma.cu serves this attention (the library decides by the same sizes)."""
+        k = self.k_cache
+        return (self.values_in_keys and self.num_kv_heads == 1 and 128 < self.head_dim <= 576 and k is not None
+                and k.dtype == torch.bfloat16 and self.head_dim % 8 == 0 and self.v_head_dim % 8 == 0
+                and self.v_head_dim <= 512 and self.slopes is None and self.rel is None and int(self.page_size) % 64 == 0)
 
     def forward(self, qkv: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         from compactor_vllm import _native as N
@@ -341,7 +353,7 @@ class BiasedChunkAttention(nn.Module):
             N.check(lib.cvllm_bias_attn_decode_dist(
                 N.ptr(q), N.ptr(self.k_cache), N.ptr(v_cache), *table, N.ptr(ctx.positions_i32),
                 N.ptr(ctx.batch_mapping), N.ptr(self.slopes), self.chunk, *dist, int(self.sink), N.ptr(self.sink_logits),
-                self.scale, N.ptr(out), o_stride, T, H, G, D, Dv, RESERVED_BATCH, splits, N.ptr(ws), ws.numel() if ws is not None else 0, v_stride, code,
+                self.scale, N.ptr(out), o_stride, T, H, G, D, Dv, self.k_cache.shape[0], RESERVED_BATCH, splits, N.ptr(ws), ws.numel() if ws is not None else 0, v_stride, code,
                 N.stream(dev)), "cvllm_bias_attn_decode")
         if keep != Dv:
             out = out.view(T, H, Dv)[:, :, :keep]

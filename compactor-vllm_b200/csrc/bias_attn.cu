@@ -1107,6 +1107,15 @@ int cvllm_launch_prefill_bias(const void* q, const void* k_cache, const void* v_
                               int PS, int NLP, int max_seqlen_q, float scale, int chunk, int window, int keep, int sink,
                               const float* sink_logits, int64_t o_stride, cudaStream_t st);
 
+// latent_attn_umma.cu: tcgen05 / TMEM / TMA for one key/value head whose values are columns of its key rows, 16-bit
+bool cvllm_latent_attn_umma_serves(int D, int Dv, int page_size, int64_t out_stride, const void* q, const void* cache,
+                                   const void* out);
+int cvllm_launch_latent_attn_umma(const void* q, const void* cache, int64_t cache_rows, void* out, int64_t o_stride,
+                                  const int32_t* seq_start, const int32_t* cu_q, const int32_t* batch_mapping,
+                                  const int32_t* table, int64_t table_stride_slot, int B, int tokens, int max_new, int H,
+                                  int D, int Dv, int PS, float scale, int chunk, int window, int keep, int sink,
+                                  const float* sink_logits, int splits, float* part, int reserved_slot, cudaStream_t st);
+
 static int check_dtype(int dtype) { return dtype == CVLLM_BF16 || dtype == CVLLM_F32; }
 
 static int rope_qknorm_store_impl(const double* inv_freq, int rot_dims, int norm, const void* qkv, int64_t qkv_stride, const float* q_weight, const float* k_weight,
@@ -1225,13 +1234,21 @@ extern "C" int cvllm_bias_attn_varlen_dist(const void* q, const void* k_cache, c
 #define CVLLM_GO(T, BN) \
   return dispatch_dvc<T, BN>(dvc, q, c, cu_seqlens_q, seq_start, batch_mapping, slopes, chunk, db, fs, sink_logits, scale, out, \
                              out_stride, B, max_new, H, G, D, Dv, st)
-  const int path = test_options().bias_attn_fma.load();   // 0 product, 1 fp32 FMA kernel, 2 no tcgen05 kernel
+  // 0 product, 1 fp32 FMA kernel, 2 no tcgen05 kernel, 3 the latent tcgen05 kernel wherever it serves
+  const int path = test_options().bias_attn_fma.load();
   if (dtype == CVLLM_BF16 && D == 128 && Dv == 128 && v_stride == Dv && page_size % 128 == 0 && (H / G) % 2 == 0 &&
       path == 0 && dist_bias == nullptr && out_stride % 8 == 0 &&
       table_stride_head == pages_per_head && table_stride_slot == (int64_t)G * pages_per_head && cache_rows > 0)
     return cvllm_launch_prefill_bias(q, k_cache, v_cache, cache_rows, out, seq_start, slopes, page_table,
                                      batch_mapping, cu_seqlens_q, B, total_tokens, H, G, page_size, pages_per_head,
                                      max_new, scale, chunk, window, keep_first, sink, sink_logits, out_stride, st);
+  // rows wider than the mma.sync kernel's, or asked for (path 3)
+  if (dtype == CVLLM_BF16 && G == 1 && v_cache == k_cache && v_stride == D && slopes == nullptr && dist_bias == nullptr &&
+      cache_rows > 0 && ((path == 0 && D > 128) || path == 3) &&
+      cvllm_latent_attn_umma_serves(D, Dv, page_size, out_stride, q, k_cache, out))
+    return cvllm_launch_latent_attn_umma(q, k_cache, cache_rows, out, out_stride, seq_start, cu_seqlens_q, batch_mapping,
+                                         page_table, table_stride_slot, B, total_tokens, max_new, H, D, Dv, page_size,
+                                         scale, chunk, window, keep_first, sink, sink_logits, 1, nullptr, -1, st);
   if (dtype == CVLLM_BF16 && D % 16 == 0 && Dv % 8 == 0 && D <= 128 && Dv <= 128 && path != 1 &&
       v_stride % vec == 0 && aligned16(k_cache) && aligned16(v_cache) && out_stride % 2 == 0 &&
       reinterpret_cast<uintptr_t>(out) % 4 == 0) {
@@ -1260,7 +1277,7 @@ extern "C" int cvllm_bias_attn_decode(const void* q, const void* k_cache, const 
                                       size_t workspace_bytes, int64_t v_stride, int dtype, cvllm_stream_t stream) {
   return cvllm_bias_attn_decode_dist(q, k_cache, v_cache, page_table, table_stride_slot, table_stride_head, page_size,
                                      positions, batch_mapping, slopes, chunk, 0, 0, nullptr, 0, sink, sink_logits, scale,
-                                     out, 0, B, H, G, D, Dv, reserved_slot, splits, workspace, workspace_bytes, v_stride,
+                                     out, 0, B, H, G, D, Dv, 0, reserved_slot, splits, workspace, workspace_bytes, v_stride,
                                      dtype, stream);
 }
 
@@ -1270,7 +1287,7 @@ extern "C" int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, c
                                            const int32_t* batch_mapping, const float* slopes, int chunk, int window,
                                            int keep_first, const float* dist_bias, int dist_rows, int sink,
                                            const float* sink_logits, float scale, void* out, int64_t out_stride, int B,
-                                           int H, int G, int D, int Dv,
+                                           int H, int G, int D, int Dv, int64_t cache_rows,
                                            int reserved_slot, int splits, float* workspace, size_t workspace_bytes,
                                            int64_t v_stride, int dtype, cvllm_stream_t stream) {
   CVLLM_CHECK_ARG(B >= 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && Dv > 0 && chunk >= 0 && splits >= 1);
@@ -1286,6 +1303,24 @@ extern "C" int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, c
   if (v_stride == 0) v_stride = Dv;
   auto st = static_cast<cudaStream_t>(stream);
   const PagedKV c = make_paged(k_cache, v_cache, page_table, table_stride_slot, table_stride_head, page_size, v_stride);
+  const int path = test_options().bias_attn_fma.load();   // as for portions
+  if (dtype == CVLLM_BF16 && G == 1 && v_cache == k_cache && v_stride == D && slopes == nullptr && dist_bias == nullptr &&
+      cache_rows > 0 && ((path == 0 && D > 128) || path == 3) &&
+      cvllm_latent_attn_umma_serves(D, Dv, page_size, out_stride, q, k_cache, out)) {
+    if (splits > 1 && (workspace == nullptr || workspace_bytes < sizeof(float) * (size_t)B * H * splits * (2 + Dv))) {
+      set_last_error("decode workspace too small");
+      return CVLLM_E_WORKSPACE;
+    }
+    const int rc = cvllm_launch_latent_attn_umma(q, k_cache, cache_rows, out, out_stride, positions, nullptr,
+                                                 batch_mapping, page_table, table_stride_slot, B, B, 1, H, D, Dv,
+                                                 page_size, scale, chunk, window, keep_first, sink, sink_logits, splits,
+                                                 workspace, reserved_slot, st);
+    if (rc != CVLLM_OK || splits == 1) return rc;
+    bias_attn_decode_merge_kernel<__nv_bfloat16><<<B * H, 128, 0, st>>>(
+        workspace, sink ? 1.f : 0.f, sink_logits, H, static_cast<__nv_bfloat16*>(out), out_stride, Dv, splits);
+    CVLLM_CHECK_LAUNCH();
+    return CVLLM_OK;
+  }
   if (D % 8 == 0 && Dv % 8 == 0 && D <= 256 && Dv <= 256 && v_stride % 8 == 0 && aligned16(k_cache) &&
       aligned16(v_cache)) {
     if (splits > 1) {

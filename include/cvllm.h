@@ -67,7 +67,8 @@ uint64_t cvllm_launch_count(void);
  *   "grs_probe" mask         timing probes of cvllm_gemm_allreduce (results are wrong on purpose: 1 no TMA loads,
  *                            2 no UMMA, 4 no stores, 8 no reduce, 16 no L2 hints)
  *   "bias_attn_fma" 0|1|2    bfloat16 portions of cvllm_bias_attn_varlen: 0 product choice, 1 the fp32 FMA kernel,
- *                            2 mma.sync also where the tcgen05 kernel would serve (A/B)
+ *                            2 mma.sync also where the tcgen05 kernel would serve (A/B), 3 the tcgen05 kernel for latent
+ *                            rows wherever it serves (portions and decode)
  *   "ssm_segment" n          tokens per segment of cvllm_ssm_scan (0 = the product's choice; tests use short segments)
  *   "grs_debug_host_ptr" p   pinned host buffer (64 words per CTA) for cvllm_gemm_allreduce's timeout records
  * Returns CVLLM_E_ARG for an unknown name. */
@@ -536,7 +537,10 @@ int cvllm_bias_attn_decode(const void* q, const void* k_cache, const void* v_cac
  * table, so any rule from distance to bias (buckets of a smaller learned table) is served.  keep_first > 0: the
  * sequence's first keep_first positions stay visible to every later query whatever window and chunk say.  out_stride:
  * elements between the outputs of neighbouring tokens (0 = H * Dv).  A bias table runs on the mma.sync and fp32 FMA
- * kernels only; windows and kept tokens on all of them. */
+ * kernels only; windows and kept tokens on all of them.
+ * cache_rows (decode; 0 = unknown) = rows of k_cache.  bfloat16 rows of 128 < D <= 576 numbers whose values are columns
+ * of the keys (G = 1, v_cache = k_cache, v_stride = D, Dv <= 512, sizes multiples of 8, pages multiples of 64) take the
+ * tcgen05 kernel of csrc/latent_attn_umma.cu in both entry points; its `splits` count key splits likewise. */
 int cvllm_bias_attn_varlen_dist(const void* q, const void* k_cache, const void* v_cache, const int32_t* page_table,
                                 int64_t table_stride_slot, int64_t table_stride_head, int page_size,
                                 const int32_t* cu_seqlens_q, const int32_t* seq_start, const int32_t* batch_mapping,
@@ -549,8 +553,12 @@ int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, const void* 
                                 const int32_t* positions, const int32_t* batch_mapping, const float* slopes, int chunk,
                                 int window, int keep_first, const float* dist_bias, int dist_rows, int sink,
                                 const float* sink_logits, float scale, void* out, int64_t out_stride, int B, int H,
-                                int G, int D, int Dv, int reserved_slot, int splits, float* workspace, size_t workspace_bytes, int64_t v_stride, int dtype,
+                                int G, int D, int Dv, int64_t cache_rows, int reserved_slot, int splits, float* workspace, size_t workspace_bytes, int64_t v_stride, int dtype,
                                 cvllm_stream_t stream);
+
+/* How many CTAs of the latent tcgen05 kernel have given up on a wait since the library was loaded (their outputs are
+ * NaN); synchronises. */
+int cvllm_latent_attn_aborts(int* count);
 
 /* ------------------------------------------------------------------------
  * Latent attention (csrc/latent_attn.cu): the steps around attention in the latent space.  The cache row of a token

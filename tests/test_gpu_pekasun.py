@@ -338,6 +338,53 @@ def test_latent_rows_with_a_window_and_sinks(case, window):
         assert (got - want).abs().max() < (3e-2 if dtype == torch.bfloat16 else 2e-4)
 
 
+# (heads, D, Dv, page size, option): wide rows take the kernel by themselves, narrow ones when it is asked for
+WIDE = {"576": (5, 576, 512, 64, 0), "576_heads_of_48": (48, 576, 512, 128, 0), "partial_chunks": (3, 200, 136, 64, 0),
+        "130_heads": (130, 144, 80, 64, 0), "two_slices_of_320": (16, 384, 320, 192, 0), "whole_row": (2, 136, 136, 64, 0),
+        "narrow": (7, 80, 64, 64, 3), "one_chunk": (33, 64, 64, 128, 3)}
+
+
+@pytest.mark.parametrize("name", sorted(WIDE))
+@pytest.mark.parametrize("window,keep", [(0, 0), (33, 0), (150, 0), (64, 70), (1, 2)])
+@pytest.mark.parametrize("threshold", [-1.0, 0.0])
+def test_wide_latent_rows_on_tensor_cores(name, window, keep, threshold):
+    """csrc/latent_attn_umma.cu: one planted key per sequence at the edges of window and kept tokens, sinks of very
+    different size, portions and decoding with one and several key splits; threshold 0 rescales at every growing maximum."""
+    import ctypes
+
+    from compactor_vllm import _native as N
+
+    H, D, Dv, ps, option = WIDE[name]
+    scale = D ** -0.5
+    L = 250 if D > 300 else 400
+    seqs = []
+    for i, (n, at) in enumerate(((L, [keep]), (L - 11, [keep - 1 if keep else 1, 60]), (L // 3, [20]))):
+        q, k, _ = planted(n, H, 1, D, Dv, 40 + i, at)
+        seqs.append((q, k, k[..., :Dv]))
+    m = make_module(H, 1, D, Dv, scale, window=window, keep_first=keep, values_in_keys=True, sink=True, learned_sink=True)
+    g = torch.Generator().manual_seed(3)
+    sink = 4 * torch.randn(H, generator=g)
+    with torch.no_grad():
+        m.sink_logits.copy_(sink)
+    N.set_test_option("prefill_threshold", threshold)
+    try:
+        for starts in ([0, 1, 2], [L - 70, L - 13, L // 3 - 1]):
+            want = dense_reference(starts, seqs, window, keep, scale, sink.double())
+            got = paged_attention(m, torch.bfloat16, seqs, starts, ps, option, values_in_keys=True, wide_out=starts[0] == 0)
+            assert (got - want).abs().max() < 3e-2, (starts, (got - want).abs().max())
+        want = dense_reference([len(s[0]) - 1 for s in seqs], seqs, window, keep, scale, sink.double())
+        for splits in (1, 2, 5):
+            m.decode_splits = lambda *_: splits
+            got = paged_attention(m, torch.bfloat16, seqs, None, ps, option, decode=True, values_in_keys=True,
+                                  wide_out=splits == 2)
+            assert (got - want).abs().max() < 3e-2, splits
+    finally:
+        N.set_test_option("prefill_threshold", -1.0)
+    count = ctypes.c_int(-1)
+    N.check(N.lib().cvllm_latent_attn_aborts(ctypes.byref(count)), "aborts")
+    assert count.value == 0
+
+
 # ------------------------------------------------------------------------------------------------------ single layers
 MIXER_CASES = {
     "attention": (attn(4, 2, 12, 10, 7, 3), None),
@@ -658,6 +705,7 @@ OTHER_SIZES = {
     "wide_heads": [(attn(2, 1, 128, 128, 30, 2), None), (latent(2, 64, 64, 128, 192, 26), dense(32))],
     "key_of_72_value_of_136": [(attn(2, 2, 72, 136, 25, 9), None), (latent(3, 40, 24, 8, 136, 25), None)],
     "rows_of_576": [(latent(2, 128, 64, 128, 512, 21), dense(8))],
+    "wide_latent_pages": [(latent(6, 32, 32, 24, 160, 21), dense(8)), (attn(2, 1, 64, 64, 9, 2), None), 0],
     "attention_alone_no_mlp": [(attn(2, 1, 8, 8, 5, 1), None), 0, 0],
 }
 
@@ -669,7 +717,7 @@ def test_other_sizes(name, dtype):
 
     width = {"everything_one": 6, "wide_heads": 128}.get(name, 40)
     c = model_cfg(OTHER_SIZES[name], vocab=37, width=width, eps=3e-6)
-    r, t = build(c, dtype, pages=10)
+    r, t = build(c, dtype, pages=4 if "wide_latent" in name else 10, page_size=64 if "wide_latent" in name else 16)
     toks = tokens(50, 37, 9)
     want = O.forward(c, t, toks)
     for sizes in ([50], [9, 2, 1]):
