@@ -270,20 +270,23 @@ class BiasedChunkAttention(nn.Module):
         if self.window:
             keys = min(keys, self.window)
         keys = min(keys + self.keep_first, max_keys)
-        if self.wide_latent_rows:
-            # the tcgen05 kernel for wide latent rows: a CTA per (128 heads, 256 value columns, split), tiles of 64 keys
+        if self.latent_decode_kernel:
+            # a CTA per (128 heads, 256 value columns, split): one wave of an SM each, at least four tiles of 64 keys a
+            # split (measured at 32 heads, 8 sequences, rows of 128: 1024 keys 17 / 19 / 22 us with 4 / 8 / 16 splits,
+            # 4096 keys 34 / 27 / 26 us; rows of 576: 32 / 36 / 52 and 80 / 62 / 77 us)
             ctas = max(batch * -(-self.num_heads // 128) * -(-self.v_head_dim // 256), 1)
-            return int(max(1, min(148 // ctas, keys // 128, 64)))
+            return int(max(1, min(148 // ctas, keys // 256, 64)))
         ctas = max(batch * self.num_kv_heads * -(-(self.num_heads // self.num_kv_heads) // 4), 1)
         one_wave = min(296 // ctas, keys // 128)
         several = min(2048 // ctas, keys // 1024)
         return int(max(1, min(max(one_wave, several), 64)))
 
     @property
-    def wide_latent_rows(self) -> bool:
-        """Whether csrc/latent_attn_umma.cu serves this attention (the library decides by the same sizes)."""
+    def latent_decode_kernel(self) -> bool:
+        """Whether csrc/latent_attn_umma.cu serves this attention's decode steps (the library decides by the same
+        sizes)."""
         k = self.k_cache
-        return (self.values_in_keys and self.num_kv_heads == 1 and 128 < self.head_dim <= 576 and k is not None
+        return (self.values_in_keys and self.num_kv_heads == 1 and self.num_heads >= 8 and self.head_dim <= 576 and k is not None
                 and k.dtype == torch.bfloat16 and self.head_dim % 8 == 0 and self.v_head_dim % 8 == 0
                 and self.v_head_dim <= 512 and self.slopes is None and self.rel is None and int(self.page_size) % 64 == 0)
 

@@ -1242,9 +1242,9 @@ extern "C" int cvllm_bias_attn_varlen_dist(const void* q, const void* k_cache, c
     return cvllm_launch_prefill_bias(q, k_cache, v_cache, cache_rows, out, seq_start, slopes, page_table,
                                      batch_mapping, cu_seqlens_q, B, total_tokens, H, G, page_size, pages_per_head,
                                      max_new, scale, chunk, window, keep_first, sink, sink_logits, out_stride, st);
-  // rows wider than the mma.sync kernel's, or asked for (path 3)
+  // latent rows that the pipeline above has not taken
   if (dtype == CVLLM_BF16 && G == 1 && v_cache == k_cache && v_stride == D && slopes == nullptr && dist_bias == nullptr &&
-      cache_rows > 0 && ((path == 0 && D > 128) || path == 3) &&
+      cache_rows > 0 && (path == 0 || path == 3) &&
       cvllm_latent_attn_umma_serves(D, Dv, page_size, out_stride, q, k_cache, out))
     return cvllm_launch_latent_attn_umma(q, k_cache, cache_rows, out, out_stride, seq_start, cu_seqlens_q, batch_mapping,
                                          page_table, table_stride_slot, B, total_tokens, max_new, H, D, Dv, page_size,
@@ -1305,7 +1305,7 @@ extern "C" int cvllm_bias_attn_decode_dist(const void* q, const void* k_cache, c
   const PagedKV c = make_paged(k_cache, v_cache, page_table, table_stride_slot, table_stride_head, page_size, v_stride);
   const int path = test_options().bias_attn_fma.load();   // as for portions
   if (dtype == CVLLM_BF16 && G == 1 && v_cache == k_cache && v_stride == D && slopes == nullptr && dist_bias == nullptr &&
-      cache_rows > 0 && ((path == 0 && D > 128) || path == 3) &&
+      cache_rows > 0 && ((path == 0 && H >= 8) || path == 3) &&
       cvllm_latent_attn_umma_serves(D, Dv, page_size, out_stride, q, k_cache, out)) {
     if (splits > 1 && (workspace == nullptr || workspace_bytes < sizeof(float) * (size_t)B * H * splits * (2 + Dv))) {
       set_last_error("decode workspace too small");

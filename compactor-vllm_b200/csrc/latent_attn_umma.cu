@@ -1,6 +1,7 @@
 // Attention over latent rows on tcgen05 / TMEM / TMA: ONE key/value head whose values are the first Dv columns of its key
-// rows, for rows wider than the 128 numbers prefill_attn_bias.cu serves (D <= 576, Dv <= 512, 16-bit storage, pages that
-// are multiples of 64 rows).  Portions of prompts and single decoded tokens run the same kernel.
+// rows (D <= 576, Dv <= 512, bfloat16 storage, pages that are multiples of 64 rows).  Portions of prompts and single
+// decoded tokens run the same kernel; portions of rows of exactly 128 numbers in pages of 128 take prefill_attn_bias.cu,
+// whose two softmax warpgroups suit them better.
 //
 // All heads read the same keys, so the M dimension of a tile is 128 consecutive rows of the [token, head] matrix of
 // queries: at 32 heads a tile is four neighbouring tokens and its rows see almost the same keys (a decoded token's

@@ -538,9 +538,10 @@ int cvllm_bias_attn_decode(const void* q, const void* k_cache, const void* v_cac
  * sequence's first keep_first positions stay visible to every later query whatever window and chunk say.  out_stride:
  * elements between the outputs of neighbouring tokens (0 = H * Dv).  A bias table runs on the mma.sync and fp32 FMA
  * kernels only; windows and kept tokens on all of them.
- * cache_rows (decode; 0 = unknown) = rows of k_cache.  bfloat16 rows of 128 < D <= 576 numbers whose values are columns
- * of the keys (G = 1, v_cache = k_cache, v_stride = D, Dv <= 512, sizes multiples of 8, pages multiples of 64) take the
- * tcgen05 kernel of csrc/latent_attn_umma.cu in both entry points; its `splits` count key splits likewise. */
+ * cache_rows (decode; 0 = unknown) = rows of k_cache.  bfloat16 rows of D <= 576 numbers whose values are columns of the
+ * keys (G = 1, v_cache = k_cache, v_stride = D, Dv <= 512, sizes multiples of 8, pages multiples of 64) take the tcgen05
+ * kernel of csrc/latent_attn_umma.cu: portions unless the one named above serves them, decode from 8 heads on; its
+ * `splits` count key splits likewise. */
 int cvllm_bias_attn_varlen_dist(const void* q, const void* k_cache, const void* v_cache, const int32_t* page_table,
                                 int64_t table_stride_slot, int64_t table_stride_head, int page_size,
                                 const int32_t* cu_seqlens_q, const int32_t* seq_start, const int32_t* batch_mapping,
