@@ -7,7 +7,7 @@ no cuSOLVER.  Each chunk's 16-bit 48x48 Gram matrix gets a symmetric
 eigendecomposition in shared memory (fp64 tridiagonal reduction + implicit QL,
 one CTA per matrix) and the score is ||x V |lambda|^-1/2||^2 — what the
 reference's SVD yields, :173-210.  A Cholesky solve is NOT equivalent: the
-rounded Gram of low-rank keys is indefinite (DESIGN 3.4).
+rounded Gram of low-rank keys is indefinite.
 """
 from __future__ import annotations
 

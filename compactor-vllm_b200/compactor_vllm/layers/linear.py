@@ -131,7 +131,7 @@ class PeerGemmAllReduce:
     `cvllm_gemm_allreduce`): tcgen05 GEMM on CTA pairs whose epilogue TMA-stores each tile into the owning rank's
     memory over NVLink (reduce-scatter), reducer warps that sum a round of rows as soon as it has landed from every
     rank and store the result into y on every rank (all-gather).  The route for PREFILL-size outputs, where the
-    separate all-reduce is 12-37 % of the layer (DESIGN 6).
+    separate all-reduce is 12-37 % of the layer.
 
     `max_rows x out_features` sizes the shared buffer (slots + y, 2 x rows x out x 2 bytes per rank).  The returned
     tensor is a view of that buffer, valid until the next call."""

@@ -230,7 +230,7 @@ __device__ __forceinline__ uint64_t umma_smem_desc(uint32_t smem_addr, uint32_t 
 }
 // The descriptor of the same operand `byte_off` bytes further: base + constant.  The 14-bit start-address field cannot
 // carry (shared memory ends below 256 KB), so the issuing thread spends one uniform add per descriptor instead of a
-// shift and two masks — it is on the critical path of every hand-off (DESIGN 3.1, tools/trace_prefill.py).
+// shift and two masks — it is on the critical path of every hand-off (tools/trace_prefill.py).
 __device__ __forceinline__ uint64_t umma_desc_add(uint64_t base, uint32_t byte_off) {
   return (base & 0xffffffff00000000ull) | (uint64_t)((uint32_t)base + (byte_off >> 4));
 }

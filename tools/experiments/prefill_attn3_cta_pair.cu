@@ -1,7 +1,7 @@
 // Causal head-sparse varlen prefill attention on CTA PAIRS (tcgen05.mma.cta_group::2).
 //
 // prefill_attn2.cu (one CTA = 128 query rows x two GQA heads, cta_group::1) spends ~85 % of its time on the issuer /
-// TMA side: with its softmax skipped altogether it still takes 6.4 of 7.5 ms at 32K (DESIGN 3.1).  Every UMMA there
+// TMA side: with its softmax skipped altogether it still takes 6.4 of 7.5 ms at 32K.  Every UMMA there
 // reads its whole B operand (the K or V tile) out of the CTA's own shared memory, and every CTA fills its own copy
 // of every K / V tile.  Here two CTAs of one TPC (a cluster of 2 along the query-tile axis) work on two consecutive
 // 128-row query tiles of the same head pair and SHARE each K / V tile: each CTA loads HALF of it (K: 64 of the

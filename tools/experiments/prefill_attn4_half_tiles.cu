@@ -1,7 +1,7 @@
 // Causal head-sparse varlen prefill attention, FOUR S streams per CTA (64-key half tiles).
 //
 // prefill_attn2.cu keeps two streams in flight per CTA (two GQA heads, one 128-key S tile each).  Its timing
-// probes (DESIGN 3.1) show the kernel is bound neither by the MUFU (exponentials removed: same time) nor by the K / V
+// probes show the kernel is bound neither by the MUFU (exponentials removed: same time) nor by the K / V
 // feed (TMA removed: same time) nor by the UMMA issue rate (the kernel's instruction mix runs at the nominal 64
 // cycles per 128x128x16 when nothing waits, tools/ubench/umma_rate.cu): with the softmax skipped AND the loads
 // skipped it still takes 6.2 of 7.4 ms.  What is left is the round trip of every hand-off — UMMA completion ->

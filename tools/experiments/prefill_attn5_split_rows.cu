@@ -18,7 +18,7 @@
 //                 named barrier per tile), lazy O rescale (only when the max grows by > 8 in log2 units), P written
 //                 back over S as packed 16-bit, epilogue O / l.  Halving the per-thread instruction stream is what
 //                 shortens the S -> P latency (1650 -> ~900 cycles per tile), which the in-kernel trace showed to be
-//                 the critical path once the issuer was lean (DESIGN 3.1).
+//                 the critical path once the issuer was lean.
 //   warp 16       TMA producer: Q0, Q1 once; K_j, V_j through ONE ring of 5 x 32 KB slots
 //                 (K0 V0 K1 V1 ...).  Prefix tiles straight from the paged cache (a 128-row tile
 //                 never crosses a page), new-token tiles from the packed k / v.
