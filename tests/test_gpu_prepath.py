@@ -162,8 +162,8 @@ def test_leverage_from_fused_sketch_is_bit_identical(lens):
 
 @pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float16])
 def test_sketch_bits_equal_the_reference_gemm(dtype):
-    """The Compactor sketch X = K.PHI is rounded to 16 bit and feeds an ill-conditioned factorisation
-   , so its BITS matter: the kernel accumulates in the natural k order of a library GEMM
+    """The Compactor sketch X = K.PHI is rounded to 16 bit and feeds an ill-conditioned factorisation,
+    so its BITS matter: the kernel accumulates in the natural k order of a library GEMM
     (mma.cuh FragNat128) and must reproduce the reference's own call — torch.matmul on the transposed
     view, compression/compactor.py:158 — at the headline shape.  Tolerates a handful of flipped ulps in case
     another cuBLAS build picks a split-K kernel (measured here: 0 of 12.6 M)."""
