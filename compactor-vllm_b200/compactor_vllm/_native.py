@@ -79,7 +79,7 @@ _SIGNATURES = {
     "cvllm_selftest_umma": (_i, [_p, _p, _p, _i, _u32, _u32, _i, _p]),
     "cvllm_sandwich_norm": (_i, [_p, _i64, _i, _p, _p, _i64, _p, _p, _i64, _i, _i, _i, _f, _f, _i, _p]),
     "cvllm_gated_act": (_i, [_p, _i64, _p, _i64, _i64, _i, _i, _f, _i, _p]),
-    "cvllm_moe_route": (_i, [_p, _i64, _p, _i, _i, _i, _i, _i, _i, _p, _p, _p]),
+    "cvllm_moe_route": (_i, [_p, _i64, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _p]),
     "cvllm_moe_combine": (_i, [_p, _p, _p, _i, _p, _i, _p, _p, _p, _i64, _p, _i64, _i, _i, _p]),
     "cvllm_expert_gemv": (_i, [_p, _i, _p, _p, _i, _p, _i, _i, _i, _i, _f, _i, _p]),
     "cvllm_latent_norm_store": (_i, [_p, _i64, _i, _i, _i, _i, _i, _p, _p, _f, _p, _p, _p, _p, _p, _p, _i64, _i, _p,
@@ -104,7 +104,7 @@ _SIGNATURES = {
                                     _i, _i, _i, _i, _i, _i, _i, _p, _sz, _i64, _i, _p]),
     "cvllm_residual_norm": (_i, [_p, _i64, _p, _i64, _i, _p, _i64, _p, _i64, _p, _p, _p, _i64, _i, _i, _i, _f, _i, _p]),
     "cvllm_embed_norm": (_i, [_p, _p, _i, _p, _p, _i, _p, _i64, _p, _i64, _i, _i, _i, _f, _p]),
-    "cvllm_pair_hash_embed": (_i, [_p, _p, _p, _p, _p, _i64, _i64, _i64, _p, _p, _i64, _i, _i, _i, _i, _p]),
+    "cvllm_pair_hash_embed": (_i, [_p, _p, _p, _p, _p, _f, _i64, _i64, _i64, _p, _p, _i64, _i, _i, _i, _i, _p]),
     "cvllm_token_shift_mix": (_i, [_p, _i64, _p, _i, _i, _p, _p, _p, _p, _p, _i, _i, _p, _i64, _i, _i, _p]),
     "cvllm_delta_rule": (_i, [_p, _i64, _p, _i64, _i, _i, _p, _p, _p, _p, _i64, _i, _p, _i, _f, _p, _p, _p, _p, _i, _i,
                               _p, _i64, _i, _i, _i, _i, _i, _i, _p]),
@@ -122,6 +122,14 @@ _SIGNATURES = {
                                   _i, _i, _p, _i64, _i, _i, _i, _i, _p]),
     "cvllm_gated_residual_norm": (_i, [_p, _i64, _i, _p, _i64, _i, _p, _i64, _p, _p, _i64, _i, _i, _i, _f, _p]),
     "cvllm_dual_norm_blend": (_i, [_p, _i64, _p, _p, _i64, _p, _p, _i64, _i, _i, _f, _f, _i, _p]),
+    "cvllm_stream_mix_norm": (_i, [_p, _i64, _i64, _p, _i64, _i, _p, _p, _p, _i64, _i64, _p, _p, _f, _p, _i64, _i, _i, _i,
+                                   _i, _f, _p]),
+    "cvllm_group_gate": (_i, [_p, _i64, _p, _i64, _p, _i64, _i64, _i, _i, _i, _p]),
+    "cvllm_row_norm_rope_store": (_i, [_p, _i64, _p, _i, _p, _p, _f, _p, _p, _p, _p, _p, _p, _i64, _i64, _i, _p,
+                                       _i, _i, _i, _i, _i, _i, _i, _p]),
+    "cvllm_lowrank_decay": (_i, [_p, _i64, _p, _p, _f, _p, _i64, _i, _i, _i, _i, _p]),
+    "cvllm_gla_scan": (_i, [_p, _i64, _i, _i, _i, _p, _i64, _f, _p, _i, _i, _p, _i, _f, _p, _p, _p, _p, _i, _i, _p, _i64,
+                            _i, _i, _i, _i, _i, _p]),
     "cvllm_unary_act": (_i, [_p, _i64, _p, _i64, _i64, _i, _i, _i, _p]),
     "cvllm_softcap": (_i, [_p, _i64, _p, _i64, _i64, _i, _f, _i, _p]),
     "cvllm_scaled_rows": (_i, [_p, _i64, _p, _p, _i, _p, _i64, _i, _i, _p]),

@@ -743,8 +743,170 @@ class PekasunConfig:
                     for l in self.layers] or [1])
 
 
+@dataclass
+class GatedLinearConfig:
+    """Gated linear attention (layers/recurrent.py `GatedLinearMixer`): `heads` heads of `dim` key and `vdim` value
+    channels, a decay sigmoid(.)^(1 / tau) per key channel.  `decay_rank` (the inner size of the decay's two-step
+    projection) is not part of config.json: a checkpoint's tensors give it; the default serves synthetic weights."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    decay_rank: int = 16
+
+    @classmethod
+    def from_json(cls, m: dict) -> "GatedLinearConfig":
+        dim = int(m["dim"])
+        c = cls(heads=int(m["heads"]), dim=dim, vdim=int(m.get("vdim", dim)), tau=float(m["tau"]),
+                decay_rank=int(m.get("decay_rank", 16)))
+        if min(c.heads, c.dim, c.vdim) < 1 or c.tau <= 0:
+            raise ValueError(f"gated linear attention: {c}")
+        return c
+
+
+@dataclass
+class RowNormAttentionConfig:
+    """Grouped-query attention with RMS norms over the whole q and k projections, a rotation of neighbouring pairs on the
+    first `rot_dims` numbers of every head with all frequencies divided by `rot_factor`, a softmax sink of score 0 and an
+    output gate per head; `kv_from` names the layer whose cached keys and values this layer reads instead of its own."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot_dims: int
+    rot_base: float
+    rot_factor: float = 1.0
+    kv_from: Optional[int] = None
+
+    @classmethod
+    def from_json(cls, m: dict) -> "RowNormAttentionConfig":
+        dim, rot, kv_from = int(m["dim"]), m.get("rot") or {}, m.get("kv_from")
+        c = cls(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), dim=dim,
+                vdim=int(m.get("vdim", dim)), scale=float(m.get("scale", dim ** -0.5)),
+                rot_dims=int(rot.get("dims", 0) or 0), rot_base=float(rot.get("base", 10000.0)),
+                rot_factor=float((rot.get("scaling") or {}).get("factor", 1.0)),
+                kv_from=None if kv_from is None else int(kv_from))
+        if c.heads % c.kv_heads or c.rot_dims % 2 or c.rot_dims > c.dim or c.rot_factor <= 0:
+            raise ValueError(f"attention: {c.heads} heads / {c.kv_heads} kv heads, rotation of {c.rot_dims} of {c.dim}, "
+                             f"factor {c.rot_factor}")
+        return c
+
+
+@dataclass
+class GroupedMoEConfig:
+    """Mixture of silu-gated experts of size `ff` (layers/moe.py, ROUTE_SIGMOID_GROUPS): `top` of `experts` per token by the
+    largest sigmoid(router logit) among the `keep` best of `groups` equal groups; the weights are the chosen scores over
+    their sum, times `route_scale`; a shared expert of size `shared_ff` (0 = none) is added, scaled by the sigmoid of one
+    logit per token."""
+    ff: int
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+    route_scale: float = 1.0
+    shared_ff: int = 0
+
+    @classmethod
+    def from_json(cls, m: Optional[dict]) -> Optional["GroupedMoEConfig"]:
+        if m is None:
+            return None
+        if m.get("kind", "moe") != "moe":
+            raise ValueError(f"unknown feed-forward kind {m.get('kind')!r}")
+        r, shared = m["router"], m.get("shared") or {}
+        g = r.get("groups") or {}
+        count = int(g.get("count", 1))
+        c = cls(ff=int(m["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), groups=count,
+                keep=int(g.get("keep", count)), route_scale=float(r.get("scale", 1.0)),
+                shared_ff=int(shared.get("ff", 0) or 0))
+        if c.groups < 1 or c.experts % c.groups or not 1 <= c.keep <= c.groups or not 1 <= c.top <= c.keep * (c.experts // c.groups):
+            raise ValueError(f"mixture of experts: top {c.top} of {c.experts} in {c.groups} groups, {c.keep} kept")
+        return c
+
+
+@dataclass
+class FikudraLayerConfig:
+    mixer_type: str                     # "gla" | "attention"
+    mixer: Any                          # GatedLinearConfig | RowNormAttentionConfig
+    mlp: Optional[GroupedMoEConfig]
+
+
+@dataclass
+class FikudraConfig:
+    """config.json of a Fikudra model: `vocab`, `width`, `streams`, `norm.eps`, `embedding` (`scale`, `bigram`: `buckets`,
+    `mul_prev`, `mul_cur`), `layers` (each with `type`, `mixer`, `mlp`).  The residual is `streams` parallel streams; every
+    sublayer reads a weighted sum of them through an RMS norm (gain 1 + w) and returns while they pass into one another."""
+    vocab_size: int
+    hidden_size: int
+    streams: int
+    rms_norm_eps: float
+    embedding_scale: float
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+    layers: List[FikudraLayerConfig]
+    torch_dtype: Any = torch.bfloat16
+    max_position_embeddings: int = 1 << 30      # rotation angles are computed from the position: no table to outgrow
+    model_type: str = "fikudra"
+    tie_word_embeddings: bool = False
+    raw: dict = field(default_factory=dict, repr=False)
+
+    MIXERS = {"gla": GatedLinearConfig, "attention": RowNormAttentionConfig}
+
+    @classmethod
+    def from_json(cls, c: dict) -> "FikudraConfig":
+        layers = []
+        for i, entry in enumerate(c["layers"]):
+            kind = entry["type"]
+            if kind not in cls.MIXERS:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            layers.append(FikudraLayerConfig(kind, cls.MIXERS[kind].from_json(entry["mixer"]),
+                                             GroupedMoEConfig.from_json(entry.get("mlp"))))
+        for i, lc in enumerate(layers):
+            j = lc.mixer.kv_from if lc.mixer_type == "attention" else None
+            if j is None:
+                continue
+            if not (0 <= j < i) or layers[j].mixer_type != "attention" or layers[j].mixer.kv_from is not None:
+                raise ValueError(f"layer {i}: kv_from {j} is not an earlier attention layer with keys of its own")
+            a, o = lc.mixer, layers[j].mixer
+            if (a.kv_heads, a.dim, a.vdim, a.rot_dims, a.rot_base, a.rot_factor) != \
+                    (o.kv_heads, o.dim, o.vdim, o.rot_dims, o.rot_base, o.rot_factor):
+                raise ValueError(f"layer {i}: head sizes or rotation differ from layer {j}'s")
+        emb = c.get("embedding") or {}
+        bg = emb.get("bigram")
+        if not bg:
+            raise ValueError("embedding.bigram is missing")
+        streams = int(c["streams"])
+        if streams < 1:
+            raise ValueError(f"streams {streams}")
+        return cls(vocab_size=int(c["vocab"]), hidden_size=int(c["width"]), streams=streams,
+                   rms_norm_eps=float((c.get("norm") or {}).get("eps", 1e-6)),
+                   embedding_scale=float(emb.get("scale", 1.0)), buckets=int(bg["buckets"]),
+                   mul_prev=int(bg["mul_prev"]), mul_cur=int(bg["mul_cur"]), layers=layers, raw=c)
+
+    # ---- the names the cache manager and the runner read from an HF config --------------------------
+    def _attn(self):
+        return [l.mixer for l in self.layers if l.mixer_type == "attention"]
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def num_key_value_heads(self) -> int:
+        return max([a.kv_heads for a in self._attn()] or [1])
+
+    @property
+    def num_attention_heads(self) -> int:
+        return max([a.heads for a in self._attn()] or [1])
+
+    @property
+    def head_dim(self) -> int:
+        return max([a.dim for a in self._attn()] or [1])
+
+
 ARCHITECTURES = {"Movolorn": MovolornConfig, "Batasun": BatasunConfig, "Fafelix": FafelixConfig,
-                 "Nununex": NununexConfig, "Pekasun": PekasunConfig}
+                 "Nununex": NununexConfig, "Pekasun": PekasunConfig, "Fikudra": FikudraConfig}
 
 
 def load_model_config(path: str):

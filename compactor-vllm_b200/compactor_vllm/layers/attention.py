@@ -114,8 +114,10 @@ def linear_bias_slopes(num_heads: int, base_exponent: float = 8.0) -> torch.Tens
     return torch.pow(torch.tensor(2.0, dtype=torch.float64), -base_exponent * h / num_heads).float()
 
 
-def pair_rotation_frequencies(dims: int, base: float, scaling: Optional[tuple] = None) -> torch.Tensor:
-    """Rotation frequencies of dims / 2 pairs as 64-bit floats: f_i = base ** (-2 i / dims).  `scaling` =
+def pair_rotation_frequencies(dims: int, base: float, scaling: Optional[tuple] = None, *,
+                              linear_factor: float = 1.0) -> torch.Tensor:
+    """Rotation frequencies of dims / 2 pairs as 64-bit floats: f_i = base ** (-2 i / dims), all divided by
+    `linear_factor` (linear scaling: positions count that much slower).  `scaling` =
     (factor, low, high, original) stretches long wavelengths: with l = 2 pi / f, f stays where l < original / high,
     becomes f / factor where l > original / low, and between the two is blended with
     s = (original / l - low) / (high - low):  (1 - s) f / factor + s f."""
@@ -132,7 +134,7 @@ def pair_rotation_frequencies(dims: int, base: float, scaling: Optional[tuple] =
             elif wavelength >= original / high:
                 s = (original / wavelength - low) / (high - low)
                 f = (1.0 - s) * f / factor + s * f
-        out.append(f)
+        out.append(f / float(linear_factor))
     return torch.tensor(out, dtype=torch.float64)
 
 
@@ -197,7 +199,10 @@ class BiasedChunkAttention(nn.Module):
     mean square.  `window` > 0: a query sees only the keys at distances 0 .. window - 1, and - `keep_first` > 0 - the
     sequence's first keep_first positions whatever their distance.  `bucket_bias` = (rows, far): a learned table `rel` [rows, H] adds rel[bucket(i - j), h] to the
     score (unscaled; buckets as in `distance_buckets`); the kernels read it spread out per distance (`dist_bias`,
-    rebuilt by `refresh_distance_bias()` whenever `rel` changes).  forward() takes the packed projection rows
+    rebuilt by `refresh_distance_bias()` whenever `rel` changes).  `row_norm`: instead of the norm per head, the whole q
+    projection (and the whole k projection) of a token is divided by its root mean square and multiplied by a weight of its
+    size, BEFORE the rotation.  `source`: another attention of the model, whose cached keys and values this one reads
+    (with its own queries); forward() then takes rows of H*D numbers and stores nothing.  forward() takes the packed projection rows
     [T, H*D + G*D + G*Dv] (row stride free): one launch rotates / norms q / k
     and writes k / v to the cache at the tokens' positions, one launch attends — the portion kernel when any
     sequence of the step brings more than one token, the decode kernel otherwise.  The step's geometry comes from the
@@ -208,8 +213,13 @@ class BiasedChunkAttention(nn.Module):
                  slopes: Optional[torch.Tensor] = None, chunk: int = 0, sink: bool = False, qk_norm: bool = False,
                  eps: float = 1e-6, values_in_keys: bool = False, learned_sink: bool = False,
                  rotation: Optional[torch.Tensor] = None, norm: bool = True, window: int = 0,
-                 bucket_bias: Optional[tuple] = None, keep_first: int = 0, value_norm: bool = False):
+                 bucket_bias: Optional[tuple] = None, keep_first: int = 0, value_norm: bool = False,
+                 row_norm: bool = False, source: Optional["BiasedChunkAttention"] = None):
         super().__init__()
+        assert not row_norm or (qk_norm and norm and not value_norm)
+        assert source is None or row_norm, "queries alone are prepared by the whole-projection norm's kernel"
+        self.row_norm = bool(row_norm)
+        self.__dict__["source"] = source          # not a submodule: its parameters belong to its own layer
         self.norm, self.value_norm = bool(norm), bool(value_norm)
         self.window, self.keep_first = int(window), int(keep_first)
         self.bias_far = 0
@@ -228,8 +238,9 @@ class BiasedChunkAttention(nn.Module):
         self.head_dim, self.v_head_dim = int(head_dim), int(v_head_dim)
         self.scale, self.chunk, self.sink, self.eps = float(scale), int(chunk), bool(sink), float(eps)
         self.register_buffer("slopes", None if slopes is None else slopes.float().contiguous(), persistent=False)
-        self.q_norm_weight = nn.Parameter(torch.ones(head_dim, dtype=torch.float32)) if qk_norm else None
-        self.k_norm_weight = nn.Parameter(torch.ones(head_dim, dtype=torch.float32)) if qk_norm else None
+        q_w, k_w = (num_heads * head_dim, num_kv_heads * head_dim) if row_norm else (head_dim, head_dim)
+        self.q_norm_weight = nn.Parameter(torch.ones(q_w, dtype=torch.float32)) if qk_norm else None
+        self.k_norm_weight = (nn.Parameter(torch.ones(k_w, dtype=torch.float32)) if qk_norm and source is None else None)
         self.k_cache: Optional[torch.Tensor] = None
         self.v_cache: Optional[torch.Tensor] = None
         self.page_table: Optional[torch.Tensor] = None
@@ -257,6 +268,9 @@ class BiasedChunkAttention(nn.Module):
 
     @property
     def qkv_width(self) -> int:
+        """Numbers of a token's row that forward() takes."""
+        if self.source is not None:
+            return self.num_heads * self.head_dim
         return (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.v_head_dim
 
     def decode_splits(self, batch: int, max_keys: int) -> int:
@@ -294,6 +308,10 @@ class BiasedChunkAttention(nn.Module):
         from compactor_vllm import _native as N
 
         ctx: Context = get_context()
+        s = self.source
+        if s is not None and self.k_cache is None:      # the source's cache views, once the cache manager has made them
+            self.k_cache, self.v_cache, self.page_table = s.k_cache, s.v_cache, s.page_table
+            self.bh_seq_lens, self.page_size = s.bh_seq_lens, s.page_size
         assert self.k_cache is not None, "KV cache must be initialized"
         T = qkv.shape[0]
         H, G, D, Dv = self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim
@@ -303,6 +321,14 @@ class BiasedChunkAttention(nn.Module):
         pt = self.page_table
         table = (N.ptr(pt), pt.stride(0), pt.stride(1), int(self.page_size))
         rot = self.inv_freq
+        if self.row_norm:
+            caches = (None, None) if s is not None else (N.ptr(self.k_cache), N.ptr(self.v_cache))
+            N.check(lib.cvllm_row_norm_rope_store(
+                N.ptr(qkv), qkv.stride(0), N.ptr(rot), 0 if rot is None else 2 * rot.numel(), N.ptr(self.q_norm_weight),
+                N.ptr(self.k_norm_weight), self.eps, N.ptr(ctx.positions_i32), N.ptr(ctx.token_slot), N.ptr(q), *caches,
+                *table, N.ptr(self.bh_seq_lens), T, H, G, D, Dv, RESERVED_BATCH, code, N.stream(dev)),
+                "cvllm_row_norm_rope_store")
+            return self.attend(q, out=out)
         N.check(lib.cvllm_rope_qknorm_store(
             N.ptr(qkv), qkv.stride(0), N.ptr(rot), 0 if rot is None else 2 * rot.numel(),
             int(self.norm) + 2 * int(self.value_norm),

@@ -48,6 +48,22 @@ def sigmoid_gate(x: torch.Tensor, gate: torch.Tensor, out: Optional[torch.Tensor
     return out
 
 
+def group_gate(x: torch.Tensor, gate: torch.Tensor, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x [T, groups * dim] times sigmoid(gate [T, groups]), one gate for each group of neighbouring columns (a head); row
+    strides free, `out` may be x."""
+    T, width = x.shape
+    groups = gate.shape[1]
+    assert gate.shape[0] == T and width % groups == 0 and x.stride(1) == 1 and gate.stride(1) == 1
+    assert gate.dtype == x.dtype
+    if out is None:
+        out = torch.empty((T, width), dtype=x.dtype, device=x.device)
+    assert out.shape == x.shape and out.stride(1) == 1 and out.dtype == x.dtype
+    N.check(N.lib().cvllm_group_gate(N.ptr(x), x.stride(0), N.ptr(gate), gate.stride(0), N.ptr(out), out.stride(0), T,
+                                     groups, width // groups, N.block_dtype_code(x.dtype), N.stream(x.device)),
+            "cvllm_group_gate")
+    return out
+
+
 def absorb_queries(q: torch.Tensor, uk: torch.Tensor, q_full: torch.Tensor) -> None:
     """q_full[t, h, :r] = q[t, h, :dim] W_uk[h] for uk [H, dim, r]: [H, T, dim] x [H, dim, r] into the first r columns of
     the attention's query rows."""

@@ -205,6 +205,60 @@ def dual_norm_blend(a: torch.Tensor, wa: torch.Tensor, b: torch.Tensor, wb: torc
     return out
 
 
+class StreamCoefficients(nn.Module):
+    """A sublayer's coefficients between `streams` parallel residual streams (fp32): what it reads (`w_in` [S]), how the
+    streams pass into one another (`mix` [from, to]) and where its output goes (`w_out` [S]); see `stream_mix_norm`."""
+
+    def __init__(self, streams: int) -> None:
+        super().__init__()
+        f32 = dict(dtype=torch.float32)
+        self.w_in = nn.Parameter(torch.full((streams,), 1.0 / streams, **f32))
+        self.mix = nn.Parameter(torch.eye(streams, **f32))
+        self.w_out = nn.Parameter(torch.ones(streams, **f32))
+
+
+def stream_mix_norm(src: torch.Tensor, streams: int, *, branch: torch.Tensor | None = None,
+                    coeff: StreamCoefficients | None = None, dst: torch.Tensor | None = None,
+                    w_in: torch.Tensor | None = None, weight: torch.Tensor | None = None, eps: float = 1e-6,
+                    gain_offset: float = 0.0, out_dtype: torch.dtype | None = None):
+    """One launch of `cvllm_stream_mix_norm` on a residual of `streams` parallel 32-bit streams.  `src` is [T, S, width],
+    or [T, width]: S equal streams (the start of the model).
+
+        branch given:  x_t <- sum_s coeff.mix[s, t] x_s + coeff.w_out[t] * branch   (all streams at once)
+        dst given:     the streams are written to it ([T, S, width]; `src` itself for an update in place)
+        weight given:  returns rms_norm(sum_t w_in[t] x_t) * (weight + gain_offset) in `out_dtype` (w_in None: plain sum)
+
+    i.e. one sublayer's way back into the streams fused with the read and the RMS norm of the next (`w_in`, `weight`)."""
+    assert src.dtype == torch.float32 and src.stride(-1) == 1
+    if src.dim() == 2:
+        (rows, width), src_row, src_stream = src.shape, src.stride(0), 0
+    else:
+        rows, s, width = src.shape
+        assert s == streams
+        src_row, src_stream = src.stride(0), src.stride(1)
+    y_code, y_stride = N.CVLLM_F32, 0
+    if branch is not None:
+        assert branch.shape == (rows, width) and branch.stride(1) == 1 and coeff is not None
+        assert coeff.mix.shape == (streams, streams) and coeff.mix.is_contiguous() and coeff.w_out.numel() == streams
+        y_code, y_stride = N.block_dtype_code(branch.dtype), branch.stride(0)
+    dst_row = dst_stream = 0
+    if dst is not None:
+        assert dst.shape == (rows, streams, width) and dst.dtype == torch.float32 and dst.stride(2) == 1
+        dst_row, dst_stream = dst.stride(0), dst.stride(1)
+    out, o_code, o_stride = None, N.CVLLM_F32, 0
+    if weight is not None:
+        assert weight.dtype == torch.float32 and weight.numel() == width and (w_in is None or w_in.numel() == streams)
+        out = torch.empty((rows, width), dtype=out_dtype or torch.float32, device=src.device)
+        o_code, o_stride = N.block_dtype_code(out.dtype), out.stride(0)
+    mix, w_out = (None, None) if branch is None else (coeff.mix, coeff.w_out)
+    rc = N.lib().cvllm_stream_mix_norm(
+        N.ptr(src), src_row, src_stream, N.ptr(branch), y_stride, y_code, N.ptr(mix), N.ptr(w_out), N.ptr(dst), dst_row,
+        dst_stream, N.ptr(w_in), N.ptr(weight), float(gain_offset), N.ptr(out), o_stride, o_code, rows, int(streams), width,
+        float(eps), N.stream(src.device))
+    N.check(rc, "cvllm_stream_mix_norm")
+    return out
+
+
 class LayerNormWeight(nn.Module):
     """Gain and bias of a layer norm kept in fp32 whatever the model dtype (the norm runs inside `residual_norm`)."""
 

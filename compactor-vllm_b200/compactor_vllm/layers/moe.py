@@ -15,7 +15,7 @@ from compactor_vllm import _native as N
 from compactor_vllm.utils.context import get_context
 
 ACT_SILU, ACT_GELU_TANH, ACT_CLAMPED_GLU = 0, 1, 2
-ROUTE_SOFTMAX_ALL, ROUTE_TOP_LOGITS, ROUTE_SIGMOID = 0, 1, 2
+ROUTE_SOFTMAX_ALL, ROUTE_TOP_LOGITS, ROUTE_SIGMOID, ROUTE_SIGMOID_GROUPS = 0, 1, 2, 3
 ACT_RELU_SQUARED = 0      # kinds of `unary_act`
 
 
@@ -37,13 +37,16 @@ def gated_act(x: torch.Tensor, kind: int, rows: int | None = None, limit: float 
 
 
 def route(logits: torch.Tensor, correction: torch.Tensor | None, top: int, groups: int, keep: int,
-          mode: int = ROUTE_SOFTMAX_ALL, experts: int | None = None):
+          mode: int = ROUTE_SOFTMAX_ALL, experts: int | None = None, scale: float = 1.0):
     """fp32 router logits [T, E] -> (idx int32 [T, top], weights fp32 [T, top]).
 
     ROUTE_SOFTMAX_ALL: s = softmax(logits); the choice is made on s + correction among the experts of the `keep` best
     of `groups` neighbour groups (a group's rank is its largest s + correction); the weights are the chosen experts'
     plain s.  ROUTE_TOP_LOGITS: the `top` largest logits are chosen, the weights are the softmax over those alone.
     ROUTE_SIGMOID: the `top` largest sigmoid(logit) are chosen, each with its own sigmoid as weight (not renormalized).
+    ROUTE_SIGMOID_GROUPS: s = sigmoid(logits); the choice as in ROUTE_SOFTMAX_ALL, with the SUM of its two largest
+    s + correction as a group's rank; the weights are the chosen experts' plain s over (their sum + 1e-20).
+    `scale` multiplies every weight.
     `experts`: only the first so many columns are router outputs (the rows may carry more, e.g. a gate logit)."""
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     T, E = logits.shape
@@ -51,7 +54,7 @@ def route(logits: torch.Tensor, correction: torch.Tensor | None, top: int, group
     idx = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     wts = torch.empty((T, top), dtype=torch.float32, device=logits.device)
     rc = N.lib().cvllm_moe_route(N.ptr(logits), logits.stride(0), N.ptr(correction), T, E, int(top), int(groups),
-                                 int(keep), int(mode), N.ptr(idx), N.ptr(wts), N.stream(logits.device))
+                                 int(keep), int(mode), float(scale), N.ptr(idx), N.ptr(wts), N.stream(logits.device))
     N.check(rc, "cvllm_moe_route")
     return idx, wts
 
@@ -99,7 +102,8 @@ class RoutedExperts(nn.Module):
     the logits), `limit` / `shared_limit` (clamps of ACT_CLAMPED_GLU), `shared_gate` (the shared expert's output is
     multiplied by the sigmoid of one more router row, so `router` has a row more than there are experts),
     `route_mode` ROUTE_SIGMOID (see `route`), `scale_inputs` (the routing weight multiplies the expert's INPUT, rounded
-    to the activations' type, instead of its output: the outputs are summed unweighted).
+    to the activations' type, instead of its output: the outputs are summed unweighted), `route_mode`
+    ROUTE_SIGMOID_GROUPS and `route_scale` (see `route`).
 
     The router runs in fp32.  Portions: (token, choice) pairs are sorted by expert; in bfloat16 (sizes multiples of 8)
     the two projections are library grouped GEMMs over the segments (`torch._grouped_mm`, segment ends on the device);
@@ -116,8 +120,10 @@ class RoutedExperts(nn.Module):
     def __init__(self, width: int, ff: int, experts: int, identity: int, top: int, groups: int, keep: int,
                  shared_ff: int, act: int = ACT_SILU, dtype: torch.dtype | None = None, *,
                  route_mode: int = ROUTE_SOFTMAX_ALL, router_bias: bool = False, limit: float = 0.0,
-                 shared_limit: float = 0.0, shared_gate: bool = False, scale_inputs: bool = False):
+                 shared_limit: float = 0.0, shared_gate: bool = False, scale_inputs: bool = False,
+                 route_scale: float = 1.0):
         super().__init__()
+        self.route_scale = float(route_scale)
         self.scale_inputs = bool(scale_inputs)
         assert not (scale_inputs and identity), "identity experts have no input to scale"
         self.width, self.ff, self.n_real, self.n_identity = width, ff, experts, identity
@@ -137,7 +143,8 @@ class RoutedExperts(nn.Module):
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         T, W = x.shape
         logits = F.linear(x.float(), self.router, self.router_bias)
-        idx, wts = route(logits, self.correction, self.top, self.groups, self.keep, self.route_mode, self.total)
+        idx, wts = route(logits, self.correction, self.top, self.groups, self.keep, self.route_mode, self.total,
+                         self.route_scale)
         shared = self.shared(x) if self.shared is not None else None
         gate = (N.ptr(logits) + 4 * self.total, logits.stride(0)) if self.shared_gate else (None, 0)
         out = torch.empty((T, W), dtype=torch.float32, device=x.device)

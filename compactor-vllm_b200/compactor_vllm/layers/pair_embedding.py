@@ -1,6 +1,6 @@
 """Token embedding plus a hashed embedding of the (previous token, token) pair.
 
-    x_t = embed[id_t] + pair[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets]
+    x_t = embed[id_t] * scale + pair[(id_(t-1) * mul_prev + id_t * mul_cur) mod buckets]
 
 A sequence's first token takes the pair table's extra last row (index `buckets`).  The previous token of a portion's
 first token is the last token of the sequence's previous step: it lives in a slot of the state pool (`prev_token`
@@ -20,8 +20,9 @@ from compactor_vllm.utils.context import get_context
 
 
 class HashedPairEmbedding(nn.Module):
-    def __init__(self, vocab: int, width: int, buckets: int, mul_prev: int, mul_cur: int):
+    def __init__(self, vocab: int, width: int, buckets: int, mul_prev: int, mul_cur: int, scale: float = 1.0):
         super().__init__()
+        self.scale = float(scale)
         self.buckets, self.mul_prev, self.mul_cur = int(buckets), int(mul_prev), int(mul_cur)
         self.tokens = nn.Embedding(vocab, width)
         self.pairs = nn.Embedding(self.buckets + 1, width)
@@ -40,6 +41,6 @@ class HashedPairEmbedding(nn.Module):
         out = torch.empty((T, W), dtype=torch.float32, device=w.device)
         N.check(N.lib().cvllm_pair_hash_embed(
             N.ptr(input_ids), N.ptr(ctx.positions_i32), N.ptr(ctx.token_slot), N.ptr(w), N.ptr(self.pairs.weight),
-            self.buckets, self.mul_prev, self.mul_cur, N.ptr(self.prev_token), N.ptr(out), out.stride(0), T, W,
+            self.scale, self.buckets, self.mul_prev, self.mul_cur, N.ptr(self.prev_token), N.ptr(out), out.stride(0), T, W,
             RESERVED_BATCH, N.block_dtype_code(w.dtype), N.stream(w.device)), "cvllm_pair_hash_embed")
         return out

@@ -27,6 +27,11 @@ starts at 0
     o = S^T q / (max(|n . q|, exp(-m')) + 1e-6),   q times dim^-1/2
 then the same unit norm, weight, sigmoid(gate).  Its W_o belongs to the caller's arrangement (`o_proj`).
 
+`GatedLinearMixer`, gated linear attention.  From the columns [q | k | v | gate | a1] of a projection of its input:
+alpha = sigmoid(W_a2 a1 + b)^(1 / tau) per head and key channel,
+    S <- diag(alpha) S + k v^T;   o = S^T q,   q times dim^-1/2
+then the unit norm per head, a weight (one vector for all heads), silu(gate) and W_o.
+
 The recurrence, decays, gates of the recurrence, unit norms and the state are fp32; projections and convolution inputs
 are in the model's type.  What a sequence carries between steps (the matrix state, the convolution's last inputs, the
 previous token's input) lives in a `MixerState`, whose tensors the state pool allocates per slot; a layer that runs
@@ -257,4 +262,56 @@ class MatrixMemoryMixer(nn.Module):
                                         N.ptr(state.max_state), g_off, GATE_SIGMOID, N.ptr(self.norm_weight), Dv,
                                         self.eps, *geom, N.ptr(ctx.batch_mapping), B, max_new, N.ptr(out),
                                         out.stride(0), H, D, Dv, RESERVED_BATCH, code, st), "cvllm_matrix_memory")
+        return self.o_proj(out)
+
+
+class GatedLinearMixer(nn.Module):
+    def __init__(self, width: int, heads: int, dim: int, vdim: int, tau: float, decay_rank: int, eps: float):
+        super().__init__()
+        self.heads, self.dim, self.vdim = int(heads), int(dim), int(vdim)
+        self.tau, self.eps = float(tau), float(eps)
+        H, D, Dv = self.heads, self.dim, self.vdim
+        self.in_parts: List[Tuple[str, int]] = [("q", H * D), ("k", H * D), ("v", H * Dv), ("g", H * Dv),
+                                                ("a1", int(decay_rank))]
+        f32 = dict(dtype=torch.float32)
+        self.a2 = nn.Linear(int(decay_rank), H * D, bias=False)
+        self.a2_bias = nn.Parameter(torch.zeros(H * D, **f32))
+        self.norm_weight = nn.Parameter(torch.ones(Dv, **f32))
+        self.o_proj = nn.Linear(H * Dv, width, bias=False)
+
+    @property
+    def in_cols(self) -> int:
+        return sum(n for _, n in self.in_parts)
+
+    def set_decay_rank(self, rank: int) -> None:
+        """The inner size of the decay projection comes with a checkpoint's tensors."""
+        self.in_parts[-1] = ("a1", int(rank))
+        self.a2 = nn.Linear(int(rank), self.heads * self.dim, bias=False, device=self.a2.weight.device,
+                            dtype=self.a2.weight.dtype)
+
+    def make_state(self) -> MixerState:
+        return MixerState({"matrix_state": ((self.heads, self.vdim, self.dim), torch.float32)})    # [value, key]
+
+    def forward(self, cols: torch.Tensor, state: MixerState) -> torch.Tensor:
+        """cols [T, >= in_cols] (row stride free; columns past in_cols are not read) -> W_o of the gated, normed read-out."""
+        ctx = get_context()
+        assert state.matrix_state is not None, "state pool must be initialized"
+        T = cols.shape[0]
+        H, D, Dv = self.heads, self.dim, self.vdim
+        dev, lib, st = cols.device, N.lib(), N.stream(cols.device)
+        code = N.block_dtype_code(cols.dtype)
+        assert cols.stride(1) == 1 and cols.shape[1] >= self.in_cols
+        geom, B, max_new = _geometry(ctx)
+        v_off = 2 * H * D
+        g_off = v_off + H * Dv
+        alpha = torch.empty((T, H * D), dtype=torch.float32, device=dev)
+        a1 = cols[:, g_off + H * Dv:]
+        N.check(lib.cvllm_lowrank_decay(N.ptr(a1), cols.stride(0), N.ptr(self.a2.weight), N.ptr(self.a2_bias),
+                                        1.0 / self.tau, N.ptr(alpha), alpha.stride(0), T, H * D,
+                                        self.a2.weight.shape[1], code, st), "cvllm_lowrank_decay")
+        out = torch.empty((T, H * Dv), dtype=cols.dtype, device=dev)
+        N.check(lib.cvllm_gla_scan(N.ptr(cols), cols.stride(0), 0, H * D, v_off, N.ptr(alpha), alpha.stride(0), D ** -0.5,
+                                   N.ptr(state.matrix_state), g_off, GATE_SILU, N.ptr(self.norm_weight), 0, self.eps,
+                                   *geom, N.ptr(ctx.batch_mapping), B, max_new, N.ptr(out), out.stride(0), H, D, Dv,
+                                   RESERVED_BATCH, code, st), "cvllm_gla_scan")
         return self.o_proj(out)

@@ -770,6 +770,110 @@ __global__ void __launch_bounds__(128) qknorm_store_vec_kernel(
   }
 }
 
+// ---------------------------------------------------------------------------------------------------------
+// q / k norm over the WHOLE projection + rotation + store, one CTA per token.  The H * D numbers of q are divided by
+// their common root mean square and multiplied by a weight of that size, the G * D numbers of k likewise; then neighbours
+// of the first rot.dims numbers of every head turn; k and v go to their cache rows.  has_kv 0: the rows hold q alone (a
+// layer that reads another layer's cache).  VEC: eight neighbours per thread (D and Dv multiples of 8, aligned rows);
+// else one pair of neighbours per thread.
+// ---------------------------------------------------------------------------------------------------------
+constexpr int kRowNormThreads = 256;
+
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
+  a = warp_sum(a);
+  b = warp_sum(b);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (lane == 0) red[warp] = make_float2(a, b);
+  __syncthreads();
+  float2 t = lane < kRowNormThreads / 32 ? red[lane] : make_float2(0.f, 0.f);
+  return make_float2(warp_sum(t.x), warp_sum(t.y));
+}
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kRowNormThreads) row_norm_rope_store_kernel(
+    const T* __restrict__ qkv, int64_t qkv_stride, const float* __restrict__ q_w, const float* __restrict__ k_w,
+    float eps, const int32_t* __restrict__ positions, const int32_t* __restrict__ token_slot, T* __restrict__ q_out,
+    T* __restrict__ k_cache, T* __restrict__ v_cache, PagedKV c, int32_t* __restrict__ bh_lens, int H, int G, int D,
+    int Dv, int reserved_slot, Rotation rot, int has_kv) {
+  extern __shared__ float rot_cs[];   // cos [dims / 2], sin [dims / 2]
+  __shared__ float2 red[kRowNormThreads / 32];
+  constexpr int V = VEC ? 8 : 2;
+  const int t = blockIdx.x;
+  const int slot = token_slot[t], pos = positions[t];
+  const bool stores = has_kv && slot != reserved_slot;
+  const int half = rot.inv_freq ? rot.dims / 2 : 0;
+  if (half > 0) fill_rotation(rot_cs, rot_cs + half, rot, pos);
+  const T* row = qkv + (int64_t)t * qkv_stride;
+  const int ch = (D + V - 1) / V;                       // pieces per head
+  const int nq = H * ch, nqk = stores ? (H + G) * ch : nq;
+  auto load = [&](int p, float (&x)[V]) {               // piece p of the q | k heads
+    const int r = p / ch, d = (p - r * ch) * V;
+    const T* src = row + (int64_t)r * D + d;
+    if constexpr (VEC) {
+      load8<T>(src, x);
+    } else {
+      x[0] = to_f<T>(src[0]);
+      x[1] = d + 1 < D ? to_f<T>(src[1]) : 0.f;
+    }
+  };
+  float sq = 0.f, sk = 0.f;
+  for (int p = threadIdx.x; p < nqk; p += kRowNormThreads) {
+    float x[V], ss = 0.f;
+    load(p, x);
+#pragma unroll
+    for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
+    if (p < nq) sq += ss;
+    else sk += ss;
+  }
+  const float2 tot = block_sum2(sq, sk, red);           // its barrier also publishes the rotation
+  const float iq = 1.0f / sqrtf(tot.x / (float)(H * D) + eps);
+  const float ik = stores ? 1.0f / sqrtf(tot.y / (float)(G * D) + eps) : 0.f;
+  for (int p = threadIdx.x; p < nqk; p += kRowNormThreads) {
+    const int r = p / ch, d = (p - r * ch) * V;
+    const bool is_q = p < nq;
+    float x[V];
+    load(p, x);
+    const float inv = is_q ? iq : ik;
+    const float* w = is_q ? q_w + (int64_t)r * D + d : k_w + (int64_t)(r - H) * D + d;
+#pragma unroll
+    for (int e = 0; e < V; ++e)
+      if (VEC || d + e < D) x[e] *= inv * w[e];
+#pragma unroll
+    for (int e = 0; e < V; e += 2) {
+      const int i = (d + e) >> 1;
+      if (i < half) {
+        const float u = x[e], v = x[e + 1];
+        x[e] = u * rot_cs[i] - v * rot_cs[half + i];
+        x[e + 1] = v * rot_cs[i] + u * rot_cs[half + i];
+      }
+    }
+    T* dst = is_q ? q_out + ((int64_t)t * H + r) * D : k_cache + cache_row(c, slot, r - H, pos) * D;
+    if constexpr (VEC) {
+      store8<T>(dst + d, x);
+    } else {
+      dst[d] = from_f<T>(x[0]);
+      if (d + 1 < D) dst[d + 1] = from_f<T>(x[1]);
+    }
+  }
+  if (!stores) return;
+  const int cv = (Dv + V - 1) / V;
+  const T* vrow = row + (int64_t)(H + G) * D;
+  for (int p = threadIdx.x; p < G * cv; p += kRowNormThreads) {
+    const int g = p / cv, d = (p - g * cv) * V;
+    const T* src = vrow + (int64_t)g * Dv + d;
+    T* dst = v_cache + cache_row(c, slot, g, pos) * Dv + d;
+    if constexpr (VEC) {
+      float x[V];
+      load8<T>(src, x);
+      store8<T>(dst, x);
+    } else {
+      dst[0] = src[0];
+      if (d + 1 < Dv) dst[1] = src[1];
+    }
+    if (d == 0 && bh_lens) atomicMax(bh_lens + slot * G + g, pos + 1);
+  }
+}
+
 template <typename T, int CH>
 __global__ void __launch_bounds__(128) bias_attn_decode_split_kernel(
     const T* __restrict__ q, PagedKV c, const int32_t* __restrict__ positions,
@@ -1188,6 +1292,44 @@ extern "C" int cvllm_rope_qknorm_store(const void* qkv, int64_t qkv_stride, cons
   return rope_qknorm_store_impl(inv_freq, rot_dims, norm, qkv, qkv_stride, q_weight, k_weight, eps, positions,
                                 token_slot, q_out, k_cache, v_cache, page_table, table_stride_slot, table_stride_head,
                                 page_size, bh_lens, T, H, G, D, Dv, reserved_slot, dtype, stream);
+}
+
+extern "C" int cvllm_row_norm_rope_store(const void* qkv, int64_t qkv_stride, const double* inv_freq, int rot_dims,
+                                         const float* q_weight, const float* k_weight, float eps,
+                                         const int32_t* positions, const int32_t* token_slot, void* q_out,
+                                         void* k_cache, void* v_cache, const int32_t* page_table,
+                                         int64_t table_stride_slot, int64_t table_stride_head, int page_size,
+                                         int32_t* bh_lens, int T, int H, int G, int D, int Dv, int reserved_slot,
+                                         int dtype, cvllm_stream_t stream) {
+  drop_stale_error();
+  const int has_kv = k_cache != nullptr;
+  CVLLM_CHECK_ARG(T >= 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && Dv > 0);
+  CVLLM_CHECK_ARG(inv_freq == nullptr || (rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= D));
+  const Rotation rot{rot_dims > 0 ? inv_freq : nullptr, rot_dims};
+  const size_t rsmem = rot.inv_freq ? sizeof(float) * (size_t)rot_dims : 0;
+  CVLLM_CHECK_SUPPORTED(rsmem <= 32 * 1024);
+  if (T == 0) return CVLLM_OK;
+  CVLLM_CHECK_ARG(qkv && q_weight && positions && token_slot && q_out && check_dtype(dtype));
+  CVLLM_CHECK_ARG(!has_kv || (k_weight && v_cache && page_table && page_size > 0));
+  auto st = static_cast<cudaStream_t>(stream);
+  const PagedKV c = make_paged(k_cache, v_cache, page_table, table_stride_slot, table_stride_head,
+                               has_kv ? page_size : 1, Dv);
+  const int64_t align = dtype == CVLLM_BF16 ? 8 : 4;
+  const bool vec = D % 8 == 0 && Dv % 8 == 0 && qkv_stride % align == 0 && aligned16(qkv) && aligned16(q_out) &&
+                   aligned16(k_cache) && aligned16(v_cache);
+#define CVLLM_ROWNORM(TT, VV)                                                                                        \
+  row_norm_rope_store_kernel<TT, VV><<<T, kRowNormThreads, rsmem, st>>>(                                             \
+      static_cast<const TT*>(qkv), qkv_stride, q_weight, k_weight, eps, positions, token_slot,                       \
+      static_cast<TT*>(q_out), static_cast<TT*>(k_cache), static_cast<TT*>(v_cache), c, bh_lens, H, G, D, Dv,        \
+      reserved_slot, rot, has_kv)
+  if (dtype == CVLLM_BF16) {
+    if (vec) CVLLM_ROWNORM(__nv_bfloat16, true); else CVLLM_ROWNORM(__nv_bfloat16, false);
+  } else {
+    if (vec) CVLLM_ROWNORM(float, true); else CVLLM_ROWNORM(float, false);
+  }
+#undef CVLLM_ROWNORM
+  CVLLM_CHECK_LAUNCH();
+  return CVLLM_OK;
 }
 
 extern "C" int cvllm_bias_attn_varlen(const void* q, const void* k_cache, const void* v_cache,

@@ -165,15 +165,15 @@ __global__ void __launch_bounds__(kThreads) embed_norm_kernel(
 }
 
 // Token embedding plus a hashed embedding of the (previous token, token) pair, one CTA per token:
-//   out[t, :] = embed[id_t, :] + pair[row_t, :],   row_t = (prev_t * mul_prev + id_t * mul_cur) mod buckets,
+//   out[t, :] = embed[id_t, :] * scale + pair[row_t, :],   row_t = (prev_t * mul_prev + id_t * mul_cur) mod buckets,
 // and row_t = buckets (the table's extra last row) for a sequence's first token (position 0).  prev_t is the token
 // before t in the step when that one belongs to the same sequence (same slot, position one less), else the slot's
 // entry of prev_state (the last token of the sequence's previous step).  fp32 sum of the two rows.
 template <typename T>
 __global__ void __launch_bounds__(kThreads) pair_embed_kernel(
     const int64_t* __restrict__ ids, const int32_t* __restrict__ positions, const int32_t* __restrict__ token_slot,
-    const T* __restrict__ embed, const T* __restrict__ pair, int64_t buckets, int64_t mul_prev, int64_t mul_cur,
-    const int32_t* __restrict__ prev_state, float* __restrict__ out, int64_t o_stride, int width) {
+    const T* __restrict__ embed, const T* __restrict__ pair, float scale, int64_t buckets, int64_t mul_prev,
+    int64_t mul_cur, const int32_t* __restrict__ prev_state, float* __restrict__ out, int64_t o_stride, int width) {
   const int t = blockIdx.x;
   const int64_t id = ids[t];
   const int pos = positions[t], slot = token_slot[t];
@@ -187,7 +187,7 @@ __global__ void __launch_bounds__(kThreads) pair_embed_kernel(
   const T* e = embed + id * width;
   const T* pr = pair + prow * width;
   float* o = out + (int64_t)t * o_stride;
-  for (int i = threadIdx.x; i < width; i += kThreads) o[i] = to_f<T>(e[i]) + to_f<T>(pr[i]);
+  for (int i = threadIdx.x; i < width; i += kThreads) o[i] = fmaf(to_f<T>(e[i]), scale, to_f<T>(pr[i]));
 }
 
 // prev_state[slot] = the last token each sequence brings in this step (runs after pair_embed_kernel has read the old one)
@@ -301,10 +301,12 @@ constexpr int kRouteWarps = 4;
 // the largest group maximum of choice are struck; the `top` largest remaining choices are taken, each with
 // its plain s as weight.  mode 1: the `top` largest LOGITS are taken (lowest index first among equals) and the
 // weights are the softmax over the chosen logits alone.  mode 2: the same choice (the largest sigmoid(logit) are the
-// largest logits), each with its own sigmoid(logit) as weight, not renormalized.  Shared memory per warp: s[E], choice[E], group maxima[groups].
+// largest logits), each with its own sigmoid(logit) as weight, not renormalized.  mode 3: s = sigmoid(logits), choice =
+// s + correction; a group's rank is the SUM of its two largest choices; the weights are the chosen experts' plain s over
+// (their sum + 1e-20).  Every weight is multiplied by wscale.  Shared memory per warp: s[E], choice[E], group ranks[groups].
 __global__ void __launch_bounds__(kRouteWarps * 32) route_kernel(
     const float* __restrict__ logits, int64_t l_stride, const float* __restrict__ correction, int T, int E,
-    int top, int groups, int keep, int mode, int32_t* __restrict__ idx, float* __restrict__ wts) {
+    int top, int groups, int keep, int mode, float wscale, int32_t* __restrict__ idx, float* __restrict__ wts) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kRouteWarps + warp;
@@ -326,7 +328,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) route_kernel(
       sum += p;
       if (lane == 0) {
         idx[(int64_t)t * top + r] = e;
-        wts[(int64_t)t * top + r] = p;
+        wts[(int64_t)t * top + r] = p * wscale;
         c[e] = NAN;
       }
       __syncwarp();
@@ -334,28 +336,39 @@ __global__ void __launch_bounds__(kRouteWarps * 32) route_kernel(
     if (mode == 1 && lane < top) wts[(int64_t)t * top + lane] /= sum;   // top <= 32 in this mode (checked by the host)
     return;
   }
-  float m = -INFINITY;
-  for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
-  m = warp_max(m);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float p = expf(z[e] - m);
-    s[e] = p;
-    sum += p;
-  }
-  sum = warp_sum(sum);
-  for (int e = lane; e < E; e += 32) {
-    const float p = s[e] / sum;
-    s[e] = p;
-    c[e] = correction ? p + correction[e] : p;
+  if (mode == 3) {
+    for (int e = lane; e < E; e += 32) {
+      const float p = 1.0f / (1.0f + expf(-z[e]));
+      s[e] = p;
+      c[e] = correction ? p + correction[e] : p;
+    }
+  } else {
+    float m = -INFINITY;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+    m = warp_max(m);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      const float p = expf(z[e] - m);
+      s[e] = p;
+      sum += p;
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      const float p = s[e] / sum;
+      s[e] = p;
+      c[e] = correction ? p + correction[e] : p;
+    }
   }
   __syncwarp();
   if (groups > 1 && keep < groups) {
     const int size = E / groups;
     for (int g = lane; g < groups; g += 32) {
-      float b = -INFINITY;
-      for (int e = g * size; e < (g + 1) * size; ++e) b = fmaxf(b, c[e]);
-      gm[g] = b;
+      float b = -INFINITY, b2 = -INFINITY;    // the group's two largest choices
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        b2 = fmaxf(b2, fminf(b, c[e]));
+        b = fmaxf(b, c[e]);
+      }
+      gm[g] = mode == 3 && size > 1 ? b + b2 : b;
     }
     __syncwarp();
     // a kept group's maximum is overwritten with NaN as its mark; experts of unmarked groups are struck afterwards
@@ -370,17 +383,21 @@ __global__ void __launch_bounds__(kRouteWarps * 32) route_kernel(
       if (!isnan(gm[e / size])) c[e] = -INFINITY;
     __syncwarp();
   }
+  float chosen = 0.f;
   for (int r = 0; r < top; ++r) {
     float b;
     const int e = warp_argmax(c, E, &b);
     __syncwarp();
+    chosen += s[e];
     if (lane == 0) {
       idx[(int64_t)t * top + r] = e;
-      wts[(int64_t)t * top + r] = s[e];
+      wts[(int64_t)t * top + r] = s[e] * wscale;
       c[e] = NAN;
     }
     __syncwarp();
   }
+  if (mode == 3)
+    for (int r = lane; r < top; r += 32) wts[(int64_t)t * top + r] = s[idx[(int64_t)t * top + r]] / (chosen + 1e-20f) * wscale;
 }
 
 // out[t, :] = sum_r w[t, r] * (idx[t, r] < n_real ? y[pos[t * top + r], :] : h[t, :])  (+ s_t shared[t, :]),  fp32 sums;
@@ -500,6 +517,112 @@ __global__ void __launch_bounds__(kThreads) dual_norm_blend_kernel(const T* __re
   const float ia = scale / sqrtf(sa / (float)width + eps), ib = scale / sqrtf(sb / (float)width + eps);
   for (int i = threadIdx.x; i < width; i += kThreads)
     out[r * o_stride + i] = from_f<T>(to_f<T>(a[r * a_stride + i]) * ia * wa[i] + to_f<T>(b[r * b_stride + i]) * ib * wb[i]);
+}
+
+// One CTA per row of a model whose residual is S parallel 32-bit streams x_0 .. x_(S-1) [rows, S, width]:
+//   y != NULL:    x'_t = sum_s mix[s, t] x_s + w_out[t] y      (all t at once from the old streams; else x' = x)
+//   dst != NULL:  the new streams are written there (src itself, or elsewhere)
+//   out != NULL:  u = sum_t w_in[t] x'_t  (w_in NULL: the plain sum),  out = u / sqrt(mean(u^2) + eps) * (w + gain_offset)
+// i.e. a sublayer's way back into the streams fused with the next sublayer's read and norm.  src has strides of its own:
+// stream stride 0 reads S equal streams from one.  SMAX >= S bounds the streams a thread holds in registers (S == SMAX
+// unless GUARD).  V neighbouring columns per thread (4 needs widths, strides and bases in multiples of 16 bytes).
+template <int V>
+struct FVec {
+  float v[V];
+};
+template <int V, typename T>
+__device__ __forceinline__ FVec<V> load_cols(const T* p) {
+  FVec<V> r;
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    r.v[0] = t.x, r.v[1] = t.y, r.v[2] = t.z, r.v[3] = t.w;
+  } else if constexpr (V == 4) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack2<true>(t.x), b = unpack2<true>(t.y);
+    r.v[0] = a.x, r.v[1] = a.y, r.v[2] = b.x, r.v[3] = b.y;
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) r.v[e] = to_f<T>(p[e]);
+  }
+  return r;
+}
+template <int V, typename T>
+__device__ __forceinline__ void store_cols(T* p, const FVec<V>& r) {
+  if constexpr (V == 4 && sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack2<true>(r.v[0], r.v[1]), pack2<true>(r.v[2], r.v[3]));
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) p[e] = from_f<T>(r.v[e]);
+  }
+}
+
+constexpr int kMaxStreams = 16;
+
+template <typename TY, typename TO, int SMAX, bool GUARD, int V>
+__global__ void __launch_bounds__(kThreads) stream_mix_norm_kernel(
+    const float* src, int64_t src_row, int64_t src_stream, const TY* __restrict__ y, int64_t y_stride,
+    const float* __restrict__ mix, const float* __restrict__ w_out, float* dst, int64_t dst_row, int64_t dst_stream,
+    const float* __restrict__ w_in, const float* __restrict__ w, float gain_offset, TO* __restrict__ out,
+    int64_t o_stride, int streams, int width, float eps) {
+  extern __shared__ __align__(16) float row[];       // u [width]
+  __shared__ float red[kThreads / 32];
+  __shared__ float cm[SMAX * SMAX], co[SMAX], ci[SMAX];
+  const int64_t r = blockIdx.x;
+  const int S = GUARD ? streams : SMAX;
+  for (int i = threadIdx.x; i < S; i += kThreads) {
+    ci[i] = w_in ? w_in[i] : 1.0f;
+    if (y) co[i] = w_out[i];
+  }
+  if (y)
+    for (int i = threadIdx.x; i < S * S; i += kThreads) cm[i] = mix[i];
+  __syncthreads();
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < width; i += kThreads * V) {
+    FVec<V> x[SMAX], u;
+#pragma unroll
+    for (int s = 0; s < SMAX; ++s)
+      if (!GUARD || s < S) x[s] = load_cols<V, float>(src + r * src_row + s * src_stream + i);
+    FVec<V> yv;
+    if (y) yv = load_cols<V, TY>(y + r * y_stride + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) u.v[e] = 0.f;
+#pragma unroll
+    for (int t = 0; t < SMAX; ++t) {
+      if (GUARD && t >= S) continue;
+      FVec<V> n;
+      if (y) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) n.v[e] = co[t] * yv.v[e];
+#pragma unroll
+        for (int s = 0; s < SMAX; ++s)
+          if (!GUARD || s < S)
+#pragma unroll
+            for (int e = 0; e < V; ++e) n.v[e] = fmaf(cm[s * S + t], x[s].v[e], n.v[e]);
+      } else {
+        n = x[t];
+      }
+      if (dst) store_cols<V, float>(dst + r * dst_row + t * dst_stream + i, n);
+#pragma unroll
+      for (int e = 0; e < V; ++e) u.v[e] = fmaf(ci[t], n.v[e], u.v[e]);
+    }
+    if (out) {
+      store_cols<V, float>(row + i, u);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(u.v[e], u.v[e], ss);
+    }
+  }
+  if (out == nullptr) return;
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+  for (int i = threadIdx.x * V; i < width; i += kThreads * V) {   // every thread reads back what it wrote itself
+    FVec<V> u = load_cols<V, float>(row + i);
+    const FVec<V> g = load_cols<V, float>(w + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) u.v[e] = u.v[e] * inv * (g.v[e] + gain_offset);
+    store_cols<V, TO>(out + r * o_stride + i, u);
+  }
 }
 
 // Plain activations of one tensor.  KIND 0: relu(x)^2.
@@ -634,8 +757,8 @@ extern "C" int cvllm_embed_norm(const int64_t* ids, const void* embed, int dtype
 }
 
 extern "C" int cvllm_pair_hash_embed(const int64_t* ids, const int32_t* positions, const int32_t* token_slot,
-                                     const void* embed, const void* pair, int64_t buckets, int64_t mul_prev,
-                                     int64_t mul_cur, int32_t* prev_state, float* out, int64_t out_stride, int T,
+                                     const void* embed, const void* pair, float scale, int64_t buckets,
+                                     int64_t mul_prev, int64_t mul_cur, int32_t* prev_state, float* out, int64_t out_stride, int T,
                                      int width, int reserved_slot, int dtype, cvllm_stream_t stream) {
   drop_stale_error();
   CVLLM_CHECK_ARG(T >= 0 && width > 0 && buckets > 0);
@@ -646,12 +769,12 @@ extern "C" int cvllm_pair_hash_embed(const int64_t* ids, const int32_t* position
   if (dtype == CVLLM_BF16)
     pair_embed_kernel<__nv_bfloat16><<<T, kThreads, 0, st>>>(ids, positions, token_slot,
                                                              static_cast<const __nv_bfloat16*>(embed),
-                                                             static_cast<const __nv_bfloat16*>(pair), buckets, mul_prev,
-                                                             mul_cur, prev_state, out, out_stride, width);
+                                                             static_cast<const __nv_bfloat16*>(pair), scale, buckets,
+                                                             mul_prev, mul_cur, prev_state, out, out_stride, width);
   else
     pair_embed_kernel<float><<<T, kThreads, 0, st>>>(ids, positions, token_slot, static_cast<const float*>(embed),
-                                                     static_cast<const float*>(pair), buckets, mul_prev, mul_cur,
-                                                     prev_state, out, out_stride, width);
+                                                     static_cast<const float*>(pair), scale, buckets, mul_prev,
+                                                     mul_cur, prev_state, out, out_stride, width);
   pair_state_update_kernel<<<cdiv(T, 256), 256, 0, st>>>(ids, token_slot, prev_state, T, reserved_slot);
   CVLLM_CHECK_LAUNCHES(2);
   return CVLLM_OK;
@@ -686,10 +809,11 @@ extern "C" int cvllm_gated_act(const void* x, int64_t x_stride, void* out, int64
 }
 
 extern "C" int cvllm_moe_route(const float* logits, int64_t l_stride, const float* correction, int T, int E, int top,
-                               int groups, int keep, int mode, int32_t* idx, float* wts, cvllm_stream_t stream) {
+                               int groups, int keep, int mode, float wscale, int32_t* idx, float* wts,
+                               cvllm_stream_t stream) {
   CVLLM_CHECK_ARG(T >= 0 && E > 0 && top > 0 && top <= E && groups > 0 && keep > 0 && keep <= groups);
-  CVLLM_CHECK_ARG(mode == 0 || ((mode == 1 || mode == 2) && groups == 1 && correction == nullptr));
-  CVLLM_CHECK_SUPPORTED(mode == 0 || top <= 32);
+  CVLLM_CHECK_ARG(mode == 0 || mode == 3 || ((mode == 1 || mode == 2) && groups == 1 && correction == nullptr));
+  CVLLM_CHECK_SUPPORTED(mode == 0 || mode == 3 || top <= 32);
   if (T == 0) return CVLLM_OK;
   CVLLM_CHECK_ARG(logits && idx && wts && E % groups == 0 && keep * (E / groups) >= top);
   CVLLM_CHECK_SUPPORTED(E <= 2048);
@@ -699,7 +823,7 @@ extern "C" int cvllm_moe_route(const float* logits, int64_t l_stride, const floa
   if (smem > 48 * 1024)
     CVLLM_CHECK_CUDA(ensure_max_dyn_smem(reinterpret_cast<const void*>(route_kernel), (int)smem, mask));
   route_kernel<<<cdiv(T, kRouteWarps), kRouteWarps * 32, smem, st>>>(logits, l_stride, correction, T, E, top,
-                                                                    groups, keep, mode, idx, wts);
+                                                                    groups, keep, mode, wscale, idx, wts);
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }
@@ -858,6 +982,50 @@ extern "C" int cvllm_scaled_rows(const void* x, int64_t x_stride, const int64_t*
   else
     scaled_rows_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(x), x_stride, perm, scale, top,
                                                     static_cast<float*>(out), pairs, width);
+  CVLLM_CHECK_LAUNCH();
+  return CVLLM_OK;
+}
+
+extern "C" int cvllm_stream_mix_norm(const float* src, int64_t src_row, int64_t src_stream, const void* y,
+                                     int64_t y_stride, int y_dtype, const float* mix, const float* w_out, float* dst,
+                                     int64_t dst_row, int64_t dst_stream, const float* w_in, const float* w,
+                                     float gain_offset, void* out, int64_t o_stride, int out_dtype, int rows,
+                                     int streams, int width, float eps, cvllm_stream_t stream) {
+  drop_stale_error();
+  CVLLM_CHECK_ARG(rows >= 0 && width > 0 && streams > 0);
+  if (rows == 0) return CVLLM_OK;
+  CVLLM_CHECK_ARG(src && (y == nullptr || (mix && w_out && (y_dtype == CVLLM_BF16 || y_dtype == CVLLM_F32))));
+  CVLLM_CHECK_ARG(out == nullptr || (w != nullptr && (out_dtype == CVLLM_BF16 || out_dtype == CVLLM_F32)));
+  // a row is read before it is written only if the two tensors are the same one or do not overlap
+  CVLLM_CHECK_ARG(dst != src || (dst_row == src_row && dst_stream == src_stream && src_stream != 0));
+  CVLLM_CHECK_SUPPORTED(width <= 11776 && streams <= kMaxStreams);   // one row of u beside the coefficients in 48 KB
+  auto st = static_cast<cudaStream_t>(stream);
+  const size_t smem = (size_t)width * sizeof(float);
+  const bool yb = y && y_dtype == CVLLM_BF16, ob = out && out_dtype == CVLLM_BF16;
+  const bool vec = width % 4 == 0 && src_row % 4 == 0 && src_stream % 4 == 0 && dst_row % 4 == 0 &&
+                   dst_stream % 4 == 0 && y_stride % 8 == 0 && o_stride % 8 == 0 && aligned16(src) && aligned16(y) &&
+                   aligned16(dst) && aligned16(out) && aligned16(w);
+#define CVLLM_STREAMS(TY, TO, SM, G, V)                                                                              \
+  stream_mix_norm_kernel<TY, TO, SM, G, V><<<rows, kThreads, smem, st>>>(                                            \
+      src, src_row, src_stream, static_cast<const TY*>(y), y_stride, mix, w_out, dst, dst_row, dst_stream, w_in, w,  \
+      gain_offset, static_cast<TO*>(out), o_stride, streams, width, eps)
+#define CVLLM_STREAMS_S(TY, TO)                                              \
+  do {                                                                       \
+    if (!vec && streams <= 4) CVLLM_STREAMS(TY, TO, 4, true, 1);             \
+    else if (!vec) CVLLM_STREAMS(TY, TO, kMaxStreams, true, 1);              \
+    else if (streams == 1) CVLLM_STREAMS(TY, TO, 1, false, 4);               \
+    else if (streams == 2) CVLLM_STREAMS(TY, TO, 2, false, 4);               \
+    else if (streams == 3) CVLLM_STREAMS(TY, TO, 3, false, 4);               \
+    else if (streams == 4) CVLLM_STREAMS(TY, TO, 4, false, 4);               \
+    else if (streams <= 8) CVLLM_STREAMS(TY, TO, 8, true, 4);                \
+    else CVLLM_STREAMS(TY, TO, kMaxStreams, true, 4);                        \
+  } while (0)
+  if (yb && ob) CVLLM_STREAMS_S(__nv_bfloat16, __nv_bfloat16);
+  else if (yb) CVLLM_STREAMS_S(__nv_bfloat16, float);
+  else if (ob) CVLLM_STREAMS_S(float, __nv_bfloat16);
+  else CVLLM_STREAMS_S(float, float);
+#undef CVLLM_STREAMS_S
+#undef CVLLM_STREAMS
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }

@@ -11,6 +11,7 @@
 //                             shared key part and of every head's query part and the cache write in one launch, with
 //                             a choice of pairing and a factor on sine and cosine
 //   cvllm_sigmoid_gate        x * sigmoid(gate), element by element
+//   cvllm_group_gate          x * sigmoid(gate) with one gate per head
 // Rotation ("rotate half"): element i of a part of R numbers pairs with element i + R/2; the pair (u, v) at position
 // p becomes (u cos a - v sin a, v cos a + u sin a), a = p * inv_freq[i].  Angles and their sines are computed in
 // 64-bit (inv_freq is a 64-bit table the caller fills with base ** (-2 i / R)), norms in 32-bit.
@@ -242,6 +243,29 @@ __global__ void sigmoid_gate_kernel(const T* __restrict__ x, int64_t x_stride, c
   }
 }
 
+// one gate per group of `dim` neighbouring columns: out[t, g * dim + d] = x[t, g * dim + d] * sigmoid(gate[t, g]).
+// V columns per thread, never across a group's border (dim % V == 0).
+template <typename T, int V>
+__global__ void group_gate_kernel(const T* x, int64_t x_stride, const T* __restrict__ g, int64_t g_stride, T* out,
+                                  int64_t o_stride, int64_t rows, int groups, int dim) {
+  const int cols = groups * dim / V;
+  const int64_t total = rows * (int64_t)cols;
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = i / cols;
+    const int c = (int)(i - t * cols) * V;
+    const float f = 1.0f / (1.0f + expf(-to_f<T>(g[t * g_stride + c / dim])));
+    if constexpr (V == 8) {
+      float xv[8];
+      load8(x + t * x_stride + c, xv);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) xv[e] *= f;
+      store8(out + t * o_stride + c, xv);
+    } else {
+      out[t * o_stride + c] = from_f<T>(to_f<T>(x[t * x_stride + c]) * f);
+    }
+  }
+}
+
 }  // namespace
 }  // namespace cvllm
 
@@ -356,6 +380,29 @@ extern "C" int cvllm_sigmoid_gate(const void* x, int64_t x_stride, const void* g
     sigmoid_gate_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(x), x_stride,
                                                      static_cast<const float*>(gate), g_stride,
                                                      static_cast<float*>(out), o_stride, rows, width);
+  CVLLM_CHECK_LAUNCH();
+  return CVLLM_OK;
+}
+
+extern "C" int cvllm_group_gate(const void* x, int64_t x_stride, const void* gate, int64_t g_stride, void* out,
+                                int64_t o_stride, int64_t rows, int groups, int dim, int dtype, cvllm_stream_t stream) {
+  CVLLM_CHECK_ARG(rows >= 0 && groups > 0 && dim > 0);
+  if (rows == 0) return CVLLM_OK;
+  CVLLM_CHECK_ARG(x && gate && out && latent_dtype_ok(dtype));
+  auto st = static_cast<cudaStream_t>(stream);
+  const bool vec = dim % 8 == 0 && x_stride % 8 == 0 && o_stride % 8 == 0 && aligned16(x) && aligned16(out);
+  const int64_t total = rows * (int64_t)groups * (vec ? dim / 8 : dim);
+  const int64_t want = (total + 255) / 256, cap = (int64_t)sm_count() * 16;
+  const int grid = (int)(want < cap ? want : cap);
+#define CVLLM_GROUP_GATE(T, V)                                                                                      \
+  group_gate_kernel<T, V><<<grid, 256, 0, st>>>(static_cast<const T*>(x), x_stride, static_cast<const T*>(gate),    \
+                                                g_stride, static_cast<T*>(out), o_stride, rows, groups, dim)
+  if (dtype == CVLLM_BF16) {
+    if (vec) CVLLM_GROUP_GATE(__nv_bfloat16, 8); else CVLLM_GROUP_GATE(__nv_bfloat16, 1);
+  } else {
+    if (vec) CVLLM_GROUP_GATE(float, 8); else CVLLM_GROUP_GATE(float, 1);
+  }
+#undef CVLLM_GROUP_GATE
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }

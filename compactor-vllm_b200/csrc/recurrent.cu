@@ -6,6 +6,7 @@
 //                      (w, a per key channel, u the unit key)
 //   matrix memory      m' = max(f + m, i);  S <- e^(f + m - m') S + e^(i - m') k v^T;  n likewise with k alone;
 //                      o = S^T q / (max(|n . q|, e^(-m')) + 1e-6)        (log gates i, f per head, capped)
+//   gated linear attn. S <- diag(alpha) S + k v^T;  o = S^T q                (alpha per key channel)
 //
 // followed, inside the same kernel, by each head's unit norm (o / sqrt(mean(o^2) + eps)), a weight and a gate:
 // out = unit(o) * norm_w * silu(gate) (or sigmoid(gate)).  Also the token shift in front of the wkv projections.
@@ -15,6 +16,8 @@
 //   cvllm_wkv_scan          decays from their raw logits, the recurrence and the gated norm
 //   cvllm_general_delta     unit k, removal rates, decays, the recurrence and the gated norm
 //   cvllm_matrix_memory     capped log gates, the running maximum, the normalizer, the recurrence and the gated norm
+//   cvllm_lowrank_decay     alpha = sigmoid(W a + b)^(1 / tau), the decays of the gated linear attention
+//   cvllm_gla_scan          the recurrence and the gated norm
 //
 // Geometry of a step: cu_q [B + 1] token offsets and seq_start [B] first positions of the portions, batch_mapping [B]
 // slots of the state pool; cu_q == NULL means one token per sequence at positions[b] (decode steps, CUDA-graph
@@ -915,6 +918,370 @@ __global__ void __launch_bounds__(MAXT) matrix_memory_kernel(const T* __restrict
   if (a.VT > 1) cooperative_groups::this_cluster().sync();   // nobody leaves while its sums may still be read
 }
 
+// ---------------------------------------------------------------------------------------------------------
+// Decays of the gated linear attention.  a [T, rank] (model type), w [channels, rank] (model type), bias [channels]:
+//   z = w a + bias (fp32 sums);  alpha = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau),  fp32 [T, channels].
+// grid (channel blocks of 256, token tiles): a thread keeps its channel's weights (RANK at a time) in registers and
+// walks the tile's tokens, whose inputs lie in shared memory.
+// ---------------------------------------------------------------------------------------------------------
+constexpr int kDecayRank = 16;     // weights in registers
+constexpr int kDecayTokens = 32;   // tokens per tile
+constexpr int kDecayMaxRank = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(256) lowrank_decay_kernel(const T* __restrict__ a, int64_t a_stride,
+                                                            const T* __restrict__ w, const float* __restrict__ bias,
+                                                            float inv_tau, float* __restrict__ alpha,
+                                                            int64_t alpha_stride, int tokens, int channels, int rank) {
+  __shared__ __align__(16) float sa[kDecayTokens][kDecayMaxRank];
+  const int t0 = blockIdx.y * kDecayTokens, n = min(kDecayTokens, tokens - t0);
+  const int padded = (rank + kDecayRank - 1) / kDecayRank * kDecayRank;
+  for (int i = threadIdx.x; i < n * padded; i += 256) {
+    const int t = i / padded, r = i - t * padded;
+    sa[t][r] = r < rank ? to_f<T>(a[(int64_t)(t0 + t) * a_stride + r]) : 0.f;
+  }
+  __syncthreads();
+  const int c = blockIdx.x * 256 + threadIdx.x;
+  if (c >= channels) return;
+  const T* wr = w + (int64_t)c * rank;
+  const float b = bias[c];
+  for (int g = 0; g < n; g += 8) {
+    float z[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) z[k] = b;
+    for (int r0 = 0; r0 < rank; r0 += kDecayRank) {
+      float wv[kDecayRank];
+#pragma unroll
+      for (int r = 0; r < kDecayRank; ++r) wv[r] = r0 + r < rank ? to_f<T>(wr[r0 + r]) : 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k)
+        if (g + k < n) {
+#pragma unroll
+          for (int r = 0; r < kDecayRank; r += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(&sa[g + k][r0 + r]);
+            z[k] = fmaf(wv[r], x.x, z[k]);
+            z[k] = fmaf(wv[r + 1], x.y, z[k]);
+            z[k] = fmaf(wv[r + 2], x.z, z[k]);
+            z[k] = fmaf(wv[r + 3], x.w, z[k]);
+          }
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+      if (g + k < n) {
+        const float soft = z[k] < -20.f ? -z[k] : log1pf(expf(-z[k]));      // softplus(-z)
+        alpha[(int64_t)(t0 + g + k) * alpha_stride + c] = exp_1ulp(-soft * inv_tau);   // multiplies the state token after token
+      }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------
+// Gated linear attention.  q, k (H x D), v and the gate (H x Dv) are columns of proj (model type) at q_off, k_off (+ h * D),
+// v_off, gate_off (+ h * Dv); alpha [T, H * D] fp32.  Per head  S <- diag(alpha) S + k v^T,  o = q_scale S^T q.
+//
+// Nothing of a token waits for another token's read-out, so a thread keeps a TILE of the state: 8 rows x C value columns
+// (KS lanes of a warp hold the key rows of C columns, KS * 8 >= D; rows beyond D stay zero), and every key-sized number it
+// fetches serves C columns.  A lane's rows are two runs of four, ks * 4 and KS * 4 + ks * 4 onwards, so that neighbouring
+// lanes read neighbouring 16 bytes.  Inputs are staged as they are stored, `tok` tokens at a time, two stages deep: the
+// next stage is on its way (cp.async; plain loads where rows are not 16-byte multiples) while this one runs.  A token's
+// numbers are fetched one token ahead, and the sums over the key lanes of a token's C outputs run while the next token's
+// products do: each exchange halves the columns a lane is left with until one remains.
+// ---------------------------------------------------------------------------------------------------------
+// four numbers as they are stored; turned into floats where they are used
+template <typename T>
+struct Quad;
+template <>
+struct Quad<float> {
+  float4 v;
+  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ float2 lo() const { return make_float2(v.x, v.y); }
+  __device__ __forceinline__ float2 hi() const { return make_float2(v.z, v.w); }
+};
+template <>
+struct Quad<__nv_bfloat16> {
+  uint2 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ float2 lo() const { return unpack2<true>(v.x); }
+  __device__ __forceinline__ float2 hi() const { return unpack2<true>(v.y); }
+};
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
+}
+
+constexpr int kGlaTok = 32;     // most tokens staged at a time
+constexpr int kGlaRows = 8;     // state rows per thread
+
+struct GlaArgs {
+  int q_off, k_off, v_off;
+  int64_t proj_stride;
+  const float* alpha;
+  int64_t alpha_stride;
+  float q_scale;
+  int vec_key, vec_val;   // key- / value-sized rows move as 16-byte pieces
+  int CP;                 // staged value row: CW rounded up to 8
+};
+
+// n rows of `len` numbers (row stride `stride`) -> shared rows of `pitch` numbers
+template <typename T>
+__device__ __forceinline__ void stage_rows(T* dst, int pitch, const T* src, int64_t stride, int len, int n, bool vec) {
+  if (len <= 0) return;
+  if (vec) {
+    constexpr int E = 16 / sizeof(T);
+    TileWalk w(len / E);
+    for (; w.c < n; w.next()) cp_async16(dst + w.c * pitch + w.d * E, src + w.c * stride + w.d * E);
+  } else {
+    TileWalk w(len);
+    for (; w.c < n; w.next()) dst[w.c * pitch + w.d] = src[w.c * stride + w.d];
+  }
+}
+
+template <typename T, int KS, int C>
+__global__ void __launch_bounds__(512) gla_scan_kernel(const T* __restrict__ proj, GlaArgs ga, RecurArgs a) {
+  namespace cg = cooperative_groups;
+  constexpr int DP = KS * kGlaRows;
+  extern __shared__ __align__(16) unsigned char smraw[];
+  const int D = a.D, Dv = a.Dv, CW = a.CW, CP = ga.CP, tok = a.tok;
+  // one stage: alpha [tok][DP] fp32, q, k [tok][DP], v, gate [tok][CP]; two of them, then the outputs and the sums
+  const int stage_bytes = tok * (DP * 4 + (2 * DP + 2 * CP) * (int)sizeof(T));
+  float* so = reinterpret_cast<float*>(smraw + 2 * stage_bytes);   // [tok][CW]
+  float* part = so + tok * CW;                                     // [2][kGlaTok]
+  float* sinv = part + 2 * kGlaTok;                                // [kGlaTok]
+  const int h = blockIdx.x / a.VT, vt = blockIdx.x % a.VT, b = blockIdx.y;
+  int t0, n_new, start;
+  portion(a.g, b, t0, n_new, start);
+  if (n_new <= 0) return;               // the same for every CTA of the cluster
+  const int slot = a.g.slots[b];
+  const int c0 = vt * CW, ncol = max(0, min(CW, Dv - c0));
+  const int tid = threadIdx.x, ks = tid % KS, grp = tid / KS;
+  const int warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5;
+  const int col0 = grp * C;             // this thread's first column (of the CTA's)
+  const bool live = col0 < ncol;
+
+  // state tile: S[j][r] = rows (2 r, 2 r + 1 of the thread's eight) of column col0 + j
+  float2 S[C][kGlaRows / 2];
+  {
+    const bool from_pool = start > 0;
+#pragma unroll
+    for (int j = 0; j < C; ++j) {
+      const bool on = from_pool && col0 + j < ncol;
+      const float* p = a.state + (((int64_t)slot * a.H + h) * Dv + c0 + col0 + j) * D;
+#pragma unroll
+      for (int q4 = 0; q4 < 2; ++q4) {
+        const int i = q4 * KS * 4 + ks * 4;
+        float4 t = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (on) {
+          if ((D & 3) == 0) {
+            if (i < D) t = *reinterpret_cast<const float4*>(p + i);
+          } else {
+            if (i < D) t.x = p[i];
+            if (i + 1 < D) t.y = p[i + 1];
+            if (i + 2 < D) t.z = p[i + 2];
+            if (i + 3 < D) t.w = p[i + 3];
+          }
+        }
+        S[j][q4 * 2] = make_float2(t.x, t.y);
+        S[j][q4 * 2 + 1] = make_float2(t.z, t.w);
+      }
+    }
+  }
+  if (D != DP || ncol != CP) {   // pads: keys, queries and decays beyond D, values beyond the columns
+    for (int i = tid; i < 2 * stage_bytes / 16; i += blockDim.x)
+      reinterpret_cast<uint4*>(smraw)[i] = make_uint4(0u, 0u, 0u, 0u);
+    __syncthreads();
+  }
+  auto issue = [&](int j0, int buf) {
+    const int n = min(tok, n_new - j0);
+    unsigned char* base = smraw + buf * stage_bytes;
+    float* al = reinterpret_cast<float*>(base);
+    T* sq = reinterpret_cast<T*>(al + tok * DP);
+    T *sk = sq + tok * DP, *sv = sk + tok * DP, *sg = sv + tok * CP;
+    const T* row = proj + (int64_t)(t0 + j0) * ga.proj_stride;
+    stage_rows<float>(al, DP, ga.alpha + (int64_t)(t0 + j0) * ga.alpha_stride + h * D, ga.alpha_stride, D, n, ga.vec_key);
+    stage_rows<T>(sq, DP, row + ga.q_off + h * D, ga.proj_stride, D, n, ga.vec_key);
+    stage_rows<T>(sk, DP, row + ga.k_off + h * D, ga.proj_stride, D, n, ga.vec_key);
+    stage_rows<T>(sv, CP, row + ga.v_off + h * Dv + c0, ga.proj_stride, ncol, n, ga.vec_val);
+    stage_rows<T>(sg, CP, static_cast<const T*>(a.gate) + (int64_t)(t0 + j0) * a.gate_stride + a.gate_off + h * Dv + c0,
+                  a.gate_stride, ncol, n, ga.vec_val);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  issue(0, 0);
+  int stage = 0;
+  for (int j0 = 0; j0 < n_new; j0 += tok, ++stage) {
+    const int n = min(tok, n_new - j0);
+    if (j0 + tok < n_new) {
+      issue(j0 + tok, (stage + 1) & 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const unsigned char* base = smraw + (stage & 1) * stage_bytes;
+    const float* al = reinterpret_cast<const float*>(base);
+    const T* sq = reinterpret_cast<const T*>(al + tok * DP);
+    const T *sk = sq + tok * DP, *sv = sk + tok * DP, *sg = sv + tok * CP;
+    {
+      const int at = ks * 4, vat = live ? col0 : 0;
+      Quad<float> na[2];
+      Quad<T> nq[2], nk[2];
+      float nv[C], pend[C];
+      auto fetch = [&](int c) {
+#pragma unroll
+        for (int q4 = 0; q4 < 2; ++q4) {
+          na[q4].load(al + c * DP + q4 * KS * 4 + at);
+          nq[q4].load(sq + c * DP + q4 * KS * 4 + at);
+          nk[q4].load(sk + c * DP + q4 * KS * 4 + at);
+        }
+#pragma unroll
+        for (int j = 0; j < C; ++j) nv[j] = to_f<T>(sv[c * CP + vat + j]);
+      };
+      // sums of a token's C partial outputs over the KS key lanes; a lane ends up with C / min(C, KS) columns from `first`
+      auto finish = [&](int c) {
+        int left = C, first = 0;
+#pragma unroll
+        for (int o = 1; o < KS; o <<= 1) {
+          if (left > 1) {
+            const bool up = (ks & o) != 0;
+            left >>= 1;
+#pragma unroll
+            for (int j = 0; j < C / 2; ++j)
+              if (j < left) {
+                const float send = up ? pend[j] : pend[j + left], keep = up ? pend[j + left] : pend[j];
+                pend[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+              }
+            if (up) first += left;
+          } else {
+            pend[0] += __shfl_xor_sync(0xffffffffu, pend[0], o);
+          }
+        }
+        if (ks < C) {
+#pragma unroll
+          for (int j = 0; j < C; ++j)
+            if (j < left && col0 + first + j < ncol) so[c * CW + col0 + first + j] = pend[j] * ga.q_scale;
+        }
+      };
+      fetch(0);
+      for (int c = 0; c < n; ++c) {
+        float2 ac[4], qc[4], kc[4];
+        float vc[C], op_s[C];
+#pragma unroll
+        for (int q4 = 0; q4 < 2; ++q4) {
+          ac[2 * q4] = na[q4].lo(), ac[2 * q4 + 1] = na[q4].hi();
+          qc[2 * q4] = nq[q4].lo(), qc[2 * q4 + 1] = nq[q4].hi();
+          kc[2 * q4] = nk[q4].lo(), kc[2 * q4 + 1] = nk[q4].hi();
+        }
+#pragma unroll
+        for (int j = 0; j < C; ++j) vc[j] = nv[j];
+        if (c + 1 < n) fetch(c + 1);
+        if (c > 0) finish(c - 1);
+#pragma unroll
+        for (int j = 0; j < C; ++j) {
+          const float2 v2 = make_float2(vc[j], vc[j]);
+          float2 o2 = make_float2(0.f, 0.f);
+#pragma unroll
+          for (int r = 0; r < 4; ++r) {
+            S[j][r] = __ffma2_rn(ac[r], S[j][r], __fmul2_rn(kc[r], v2));
+            o2 = __ffma2_rn(qc[r], S[j][r], o2);
+          }
+          op_s[j] = o2.x + o2.y;
+        }
+#pragma unroll
+        for (int j = 0; j < C; ++j) pend[j] = op_s[j];
+      }
+      finish(n - 1);
+    }
+    __syncthreads();
+    // unit norm over ALL Dv columns of the head (the cluster's CTAs exchange their sums of squares), weight, gate
+    float* mine = part + (stage & 1) * kGlaTok;
+    for (int c = warp; c < n; c += warps) {
+      float ss = 0.f;
+      for (int j = lane; j < ncol; j += 32) ss = fmaf(so[c * CW + j], so[c * CW + j], ss);
+      ss = warp_sum(ss);
+      if (lane == 0) mine[c] = ss;
+    }
+    if (a.VT > 1) cg::this_cluster().sync();
+    else __syncthreads();
+    for (int c = tid; c < n; c += blockDim.x) {
+      float ss = 0.f;
+      if (a.VT > 1) {
+        cg::cluster_group cl = cg::this_cluster();
+        for (int v = 0; v < a.VT; ++v) ss += cl.map_shared_rank(mine, v)[c];
+      } else {
+        ss = mine[c];
+      }
+      sinv[c] = 1.0f / sqrtf(ss / (float)Dv + a.eps);
+    }
+    __syncthreads();
+    if (ncol > 0) {
+      T* out = static_cast<T*>(a.out);
+      TileWalk w(ncol);
+      for (; w.c < n; w.next()) {
+        const float gz = to_f<T>(sg[w.c * CP + w.d]);
+        const int col = c0 + w.d;
+        out[(int64_t)(t0 + j0 + w.c) * a.out_stride + h * Dv + col] =
+            from_f<T>(so[w.c * CW + w.d] * sinv[w.c] * a.norm_w[h * a.norm_head_stride + col] *
+                      (a.gate_kind ? sigmoid_f(gz) : silu_f(gz)));
+      }
+    }
+    __syncthreads();
+  }
+  if (slot != a.reserved_slot) {
+#pragma unroll
+    for (int j = 0; j < C; ++j) {
+      if (col0 + j >= ncol) continue;
+      float* p = a.state + (((int64_t)slot * a.H + h) * Dv + c0 + col0 + j) * D;
+#pragma unroll
+      for (int q4 = 0; q4 < 2; ++q4) {
+        const int i = q4 * KS * 4 + ks * 4;
+        const float2 lo = S[j][q4 * 2], hi = S[j][q4 * 2 + 1];
+        if ((D & 3) == 0) {
+          if (i < D) *reinterpret_cast<float4*>(p + i) = make_float4(lo.x, lo.y, hi.x, hi.y);
+        } else {
+          if (i < D) p[i] = lo.x;
+          if (i + 1 < D) p[i + 1] = lo.y;
+          if (i + 2 < D) p[i + 2] = hi.x;
+          if (i + 3 < D) p[i + 3] = hi.y;
+        }
+      }
+    }
+  }
+  if (a.VT > 1) cg::this_cluster().sync();   // nobody leaves while its sums may still be read
+}
+
+// How a (head, sequence) of the gated linear attention is laid out: KS key lanes, C columns per thread, `warps` warps per
+// CTA, VT CTAs (a cluster).  Warps work alone, so a portion wants about one per scheduler of the GPU: two columns per
+// thread instead of four while four would leave schedulers idle; CTAs of four warps, more when the step has CTAs enough.
+struct GlaShape {
+  int KS, C, VT, warps, CW, CP, tok;
+  size_t smem(size_t elem) const {
+    return 2 * (size_t)tok * ((size_t)KS * kGlaRows * (4 + 2 * elem) + 2 * (size_t)CP * elem) +
+           sizeof(float) * ((size_t)tok * CW + 3 * kGlaTok);
+  }
+};
+
+inline GlaShape gla_shape(int D, int Dv, int64_t pairs, int max_new, size_t elem) {
+  GlaShape s{};
+  s.KS = 1;
+  while (s.KS * kGlaRows < D) s.KS <<= 1;
+  auto warps_of = [&](int C) { return cdiv(Dv, 32 / s.KS * C); };
+  const int forced = test_options().gla_layout.load();   // 100 * VT + C (tests and measurements)
+  s.C = max_new > 1 && pairs * warps_of(4) < 4 * (int64_t)sm_count() ? 2 : 4;
+  if (forced > 0) s.C = forced % 100 == 2 ? 2 : 4;
+  const int w = warps_of(s.C);
+  s.VT = 1;
+  while (s.VT < 8 && s.VT * 4 < w) s.VT *= 2;
+  while (s.VT > 1 && pairs * s.VT >= 4 * (int64_t)sm_count() && cdiv(w, s.VT / 2) <= 16) s.VT /= 2;
+  if (forced > 0 && forced / 100 >= 1 && forced / 100 <= 8 && cdiv(w, forced / 100) <= 16) s.VT = forced / 100;
+  s.warps = cdiv(w, s.VT);
+  s.CW = s.warps * (32 / s.KS) * s.C;
+  s.CP = cdiv(s.CW, 8) * 8;
+  s.tok = 1;
+  while (s.tok < kGlaTok && s.tok < max_new) s.tok <<= 1;
+  while (s.tok > 1 && s.smem(elem) > 96 * 1024) s.tok >>= 1;
+  return s;
+}
+
 // How a (head, sequence) is laid out on CTAs and threads.
 struct RecurShape {
   int R, KS, VT, CW, threads, tok;
@@ -1006,6 +1373,31 @@ cudaError_t launch_clustered(K kern, dim3 grid, int threads, size_t smem, cudaSt
   cfg.attrs = attr;
   cfg.numAttrs = cluster > 1 ? 1 : 0;
   return cudaLaunchKernelEx(&cfg, kern, args...);
+}
+
+template <typename T, int KS, int C>
+int launch_gla(const GlaShape& sh, dim3 grid, cudaStream_t st, const void* proj, const GlaArgs& ga, const RecurArgs& a) {
+  static std::atomic<uint64_t> attr{0};
+  CVLLM_CHECK_CUDA(ensure_max_dyn_smem((const void*)gla_scan_kernel<T, KS, C>, 200 * 1024, attr));
+  CVLLM_CHECK_CUDA(launch_clustered(gla_scan_kernel<T, KS, C>, grid, sh.warps * 32, sh.smem(sizeof(T)), st, sh.VT,
+                                    static_cast<const T*>(proj), ga, a));
+  CVLLM_CHECK_LAUNCH();
+  return CVLLM_OK;
+}
+
+template <typename T>
+int dispatch_gla(const GlaShape& sh, dim3 grid, cudaStream_t st, const void* proj, const GlaArgs& ga, const RecurArgs& a) {
+#define CVLLM_GLA(KK) \
+  return sh.C == 2 ? launch_gla<T, KK, 2>(sh, grid, st, proj, ga, a) : launch_gla<T, KK, 4>(sh, grid, st, proj, ga, a)
+  switch (sh.KS) {
+    case 1: CVLLM_GLA(1);
+    case 2: CVLLM_GLA(2);
+    case 4: CVLLM_GLA(4);
+    case 8: CVLLM_GLA(8);
+    case 16: CVLLM_GLA(16);
+    default: CVLLM_GLA(32);
+  }
+#undef CVLLM_GLA
 }
 
 template <int R>
@@ -1237,4 +1629,56 @@ extern "C" int cvllm_matrix_memory(const void* proj, int64_t proj_stride, int q_
 #undef CVLLM_MMEM_BY_R
 #undef CVLLM_MMEM_BY_T
 #undef CVLLM_MMEM
+}
+
+extern "C" int cvllm_lowrank_decay(const void* a, int64_t a_stride, const void* w, const float* bias, float inv_tau,
+                                   float* alpha, int64_t alpha_stride, int tokens, int channels, int rank, int dtype,
+                                   cvllm_stream_t stream) {
+  drop_stale_error();
+  CVLLM_CHECK_ARG(tokens >= 0 && channels > 0 && rank > 0);
+  if (tokens == 0) return CVLLM_OK;
+  CVLLM_CHECK_ARG(a && w && bias && alpha && recur_dtype_ok(dtype));
+  CVLLM_CHECK_SUPPORTED(rank <= kDecayMaxRank && cdiv(tokens, kDecayTokens) <= 65535);
+  auto st = static_cast<cudaStream_t>(stream);
+  const dim3 grid(cdiv(channels, 256), cdiv(tokens, kDecayTokens));
+  if (dtype == CVLLM_BF16)
+    lowrank_decay_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(a), a_stride,
+                                                              static_cast<const __nv_bfloat16*>(w), bias, inv_tau, alpha,
+                                                              alpha_stride, tokens, channels, rank);
+  else
+    lowrank_decay_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(a), a_stride,
+                                                      static_cast<const float*>(w), bias, inv_tau, alpha, alpha_stride,
+                                                      tokens, channels, rank);
+  CVLLM_CHECK_LAUNCH();
+  return CVLLM_OK;
+}
+
+extern "C" int cvllm_gla_scan(const void* proj, int64_t proj_stride, int q_off, int k_off, int v_off, const float* alpha,
+                              int64_t alpha_stride, float q_scale, float* state, int gate_off, int gate_kind,
+                              const float* norm_w, int norm_head_stride, float eps, const int32_t* cu_seqlens_q,
+                              const int32_t* seq_start, const int32_t* positions, const int32_t* batch_mapping, int B,
+                              int max_new, void* out, int64_t out_stride, int H, int D, int Dv, int reserved_slot,
+                              int dtype, cvllm_stream_t stream) {
+  drop_stale_error();
+  CVLLM_CHECK_ARG(B >= 0 && max_new >= 0 && H > 0 && D > 0 && Dv > 0);
+  if (B == 0 || max_new == 0) return CVLLM_OK;
+  CVLLM_CHECK_ARG(proj && alpha && state && norm_w && batch_mapping && out && recur_dtype_ok(dtype));
+  CVLLM_CHECK_ARG(cu_seqlens_q ? seq_start != nullptr : (positions != nullptr && max_new == 1));
+  CVLLM_CHECK_SUPPORTED(D <= kMaxKeyDim && Dv <= kMaxValueDim && H <= 65535 && B <= 65535);
+  auto st = static_cast<cudaStream_t>(stream);
+  const size_t elem = dtype == CVLLM_BF16 ? 2 : 4;
+  const GlaShape sh = gla_shape(D, Dv, (int64_t)H * B, max_new, elem);
+  CVLLM_CHECK_SUPPORTED(sh.warps >= 1 && sh.warps <= 16 && sh.smem(elem) <= 200 * 1024);
+  const int E = dtype == CVLLM_BF16 ? 8 : 4;   // numbers in 16 bytes
+  const bool rows16 = aligned16(proj) && proj_stride % E == 0;
+  const int vec_key = rows16 && D % E == 0 && q_off % E == 0 && k_off % E == 0 && aligned16(alpha) &&
+                      alpha_stride % 4 == 0;
+  const int vec_val = rows16 && Dv % E == 0 && sh.CW % E == 0 && v_off % E == 0 && gate_off % E == 0;
+  const GlaArgs ga{q_off, k_off, v_off, proj_stride, alpha, alpha_stride, q_scale, vec_key, vec_val, sh.CP};
+  const RecurArgs a{{cu_seqlens_q, seq_start, positions, batch_mapping}, state, proj, proj_stride, gate_off, norm_w,
+                    norm_head_stride, eps, out, out_stride, H, D, Dv, reserved_slot, sh.KS, sh.VT, sh.CW, sh.tok,
+                    gate_kind};
+  const dim3 grid(H * sh.VT, B);
+  if (dtype == CVLLM_BF16) return dispatch_gla<__nv_bfloat16>(sh, grid, st, proj, ga, a);
+  return dispatch_gla<float>(sh, grid, st, proj, ga, a);
 }

@@ -70,6 +70,7 @@ uint64_t cvllm_launch_count(void);
  *                            2 mma.sync also where the tcgen05 kernel would serve (A/B), 3 the tcgen05 kernel for latent
  *                            rows wherever it serves (portions and decode)
  *   "ssm_segment" n          tokens per segment of cvllm_ssm_scan (0 = the product's choice; tests use short segments)
+ *   "gla_layout" n           100 * CTAs per (head, sequence) + columns per thread of cvllm_gla_scan (0 = chosen per step)
  *   "grs_debug_host_ptr" p   pinned host buffer (64 words per CTA) for cvllm_gemm_allreduce's timeout records
  * Returns CVLLM_E_ARG for an unknown name. */
 int cvllm_set_test_option(const char* name, double value);
@@ -432,13 +433,13 @@ int cvllm_embed_norm(const int64_t* ids, const void* embed, int dtype, const flo
                      int one_gain, float* resid, int64_t r_stride, void* out, int64_t o_stride, int out_dtype, int T,
                      int width, float eps, cvllm_stream_t stream);
 
-/* out[t, :] (fp32) = embed[ids[t], :] + pair[row_t, :] with row_t = (prev_t * mul_prev + ids[t] * mul_cur) mod buckets,
+/* out[t, :] (fp32) = embed[ids[t], :] * scale + pair[row_t, :] with row_t = (prev_t * mul_prev + ids[t] * mul_cur) mod buckets,
  * and row_t = buckets (the table's extra last row) where positions[t] == 0.  prev_t = ids[t - 1] when token t - 1 of
  * the step has the same slot and the position before, else prev_state[token_slot[t]]; afterwards prev_state[slot] =
  * the last token the slot brought in this step (reserved_slot excepted).  embed [V, width], pair [buckets + 1, width]. */
 int cvllm_pair_hash_embed(const int64_t* ids, const int32_t* positions, const int32_t* token_slot, const void* embed,
-                          const void* pair, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int32_t* prev_state,
-                          float* out, int64_t out_stride, int T, int width, int reserved_slot, int dtype,
+                          const void* pair, float scale, int64_t buckets, int64_t mul_prev, int64_t mul_cur,
+                          int32_t* prev_state, float* out, int64_t out_stride, int T, int width, int reserved_slot, int dtype,
                           cvllm_stream_t stream);
 
 /* Packed [gate | up] rows -> out[t, f]; kind 0: silu(gate) * up, 1: gelu_tanh(gate) * up, 2: the clamped gated unit
@@ -452,9 +453,11 @@ int cvllm_gated_act(const void* x, int64_t x_stride, void* out, int64_t o_stride
  * chosen outputs, not renormalised.  E <= 2048, E % groups == 0, keep * E / groups >= top.
  * mode 1 (groups 1, no correction, top <= 32): the `top` largest LOGITS are taken and wts is the softmax over the
  * chosen logits alone.  mode 2 (same limits): the `top` largest sigmoid(logit) are taken - the same choice - and wts
- * is each chosen output's own sigmoid(logit), not renormalised. */
+ * is each chosen output's own sigmoid(logit), not renormalised.  mode 3: s = sigmoid(logits), choice = s + correction, a
+ * group's rank is the sum of its two largest choices, and wts is the plain s of the chosen outputs over (their sum +
+ * 1e-20).  wts is multiplied by wscale in every mode. */
 int cvllm_moe_route(const float* logits, int64_t l_stride, const float* correction, int T, int E, int top,
-                    int groups, int keep, int mode, int32_t* idx, float* wts, cvllm_stream_t stream);
+                    int groups, int keep, int mode, float wscale, int32_t* idx, float* wts, cvllm_stream_t stream);
 
 /* out[t, :] = sum_r wts[t, r] * (idx[t, r] < n_real ? y[pos[t * top + r], :] : h[t, :]) + s_t * shared[t, :]
  * in fp32.  y holds one row per (token, choice) pair with a real expert, at the row pos gives (NULL: the pair's
@@ -504,6 +507,16 @@ int cvllm_rope_qknorm_store(const void* qkv, int64_t qkv_stride, const double* i
                             const int32_t* page_table, int64_t table_stride_slot, int64_t table_stride_head,
                             int page_size, int32_t* bh_lens, int T, int H, int G, int D, int Dv, int reserved_slot,
                             int dtype, cvllm_stream_t stream);
+
+/* The same step with the norm over the WHOLE projection: the H * D numbers of a token's q are divided by their common
+ * root mean square and multiplied by q_weight [H * D] (k likewise, k_weight [G * D]) BEFORE the rotation of neighbouring
+ * pairs; k and v go to the cache as they come out.  k_cache NULL: the rows hold q alone and nothing is stored. */
+int cvllm_row_norm_rope_store(const void* qkv, int64_t qkv_stride, const double* inv_freq, int rot_dims,
+                              const float* q_weight, const float* k_weight, float eps, const int32_t* positions,
+                              const int32_t* token_slot, void* q_out, void* k_cache, void* v_cache,
+                              const int32_t* page_table, int64_t table_stride_slot, int64_t table_stride_head,
+                              int page_size, int32_t* bh_lens, int T, int H, int G, int D, int Dv, int reserved_slot,
+                              int dtype, cvllm_stream_t stream);
 
 /* Portions: sequence b brings tokens cu_seqlens_q[b] .. cu_seqlens_q[b+1]-1 at positions seq_start[b] + 0, 1, ...;
  * all their keys (and every earlier one) are in the cache of slot batch_mapping[b].  out [T, H, Dv].
@@ -607,6 +620,20 @@ int cvllm_dual_norm_blend(const void* a, int64_t a_stride, const float* wa, cons
                           const float* wb, void* out, int64_t o_stride, int rows, int width, float eps, float scale,
                           int dtype, cvllm_stream_t stream);
 
+/* The residual as `streams` parallel 32-bit streams x_0 .. x_(S-1) per row, a sublayer's way back into them fused with
+ * the next sublayer's read and RMS norm, one launch:
+ *   y != NULL:   x'_t = sum_s mix[s, t] x_s + w_out[t] y   (all t at once from the old streams; y NULL: x' = x)
+ *   dst != NULL: x' is written there (element (row, s, i) at row * dst_row + s * dst_stream + i; dst == src with equal
+ *                strides updates in place, else the two must not overlap)
+ *   out != NULL: u = sum_t w_in[t] x'_t (w_in NULL: the plain sum), out = u / sqrt(mean(u^2) + eps) * (w + gain_offset)
+ * src_stream 0 reads S equal streams from one tensor.  Coefficients and weights fp32; y and out bfloat16 or float32;
+ * sums and statistics fp32.  streams <= 16, width <= 11776. */
+int cvllm_stream_mix_norm(const float* src, int64_t src_row, int64_t src_stream, const void* y, int64_t y_stride,
+                          int y_dtype, const float* mix, const float* w_out, float* dst, int64_t dst_row,
+                          int64_t dst_stream, const float* w_in, const float* w, float gain_offset, void* out,
+                          int64_t o_stride, int out_dtype, int rows, int streams, int width, float eps,
+                          cvllm_stream_t stream);
+
 /* out = act(x) element by element; kind 0: relu(x)^2. */
 int cvllm_unary_act(const void* x, int64_t x_stride, void* out, int64_t o_stride, int64_t rows, int F, int kind,
                     int dtype, cvllm_stream_t stream);
@@ -623,6 +650,11 @@ int cvllm_scaled_rows(const void* x, int64_t x_stride, const int64_t* perm, cons
 /* out[t, c] = x[t, c] * sigmoid(gate[t, c]) */
 int cvllm_sigmoid_gate(const void* x, int64_t x_stride, const void* gate, int64_t g_stride, void* out,
                        int64_t o_stride, int64_t rows, int width, int dtype, cvllm_stream_t stream);
+
+/* One gate per group of `dim` neighbouring columns (a head): out[t, g * dim + d] = x[t, g * dim + d] * sigmoid(gate[t, g]).
+ * out may be x. */
+int cvllm_group_gate(const void* x, int64_t x_stride, const void* gate, int64_t g_stride, void* out, int64_t o_stride,
+                     int64_t rows, int groups, int dim, int dtype, cvllm_stream_t stream);
 
 /* ------------------------------------------------------------------------
  * State-space mixer (csrc/ssm.cu).  A step brings sequence b the tokens cu_seqlens_q[b] .. cu_seqlens_q[b + 1] - 1 at
@@ -740,6 +772,20 @@ int cvllm_matrix_memory(const void* proj, int64_t proj_stride, int q_off, int k_
                         const int32_t* cu_seqlens_q, const int32_t* seq_start, const int32_t* positions,
                         const int32_t* batch_mapping, int B, int max_new, void* out, int64_t out_stride, int H, int D,
                         int Dv, int reserved_slot, int dtype, cvllm_stream_t stream);
+
+/* Decays of the gated linear attention: a [tokens, rank] (row stride a_stride) and w [channels, rank] of the model type,
+ * bias fp32 [channels]:  z = w a + bias,  alpha = sigmoid(z)^inv_tau,  fp32 [tokens, channels].  rank <= 256. */
+int cvllm_lowrank_decay(const void* a, int64_t a_stride, const void* w, const float* bias, float inv_tau, float* alpha,
+                        int64_t alpha_stride, int tokens, int channels, int rank, int dtype, cvllm_stream_t stream);
+
+/* Gated linear attention: q, k (H x D), v and the gate (H x Dv) are columns of proj (model type) at q_off, k_off (+ h * D),
+ * v_off, gate_off (+ h * Dv); alpha fp32 [T, H * D], a decay per key channel:
+ *   S <- diag(alpha) S + k v^T;   o = q_scale S^T q.      gate_kind 0: silu(gate), 1: sigmoid(gate). */
+int cvllm_gla_scan(const void* proj, int64_t proj_stride, int q_off, int k_off, int v_off, const float* alpha,
+                   int64_t alpha_stride, float q_scale, float* state, int gate_off, int gate_kind, const float* norm_w,
+                   int norm_head_stride, float eps, const int32_t* cu_seqlens_q, const int32_t* seq_start,
+                   const int32_t* positions, const int32_t* batch_mapping, int B, int max_new, void* out,
+                   int64_t out_stride, int H, int D, int Dv, int reserved_slot, int dtype, cvllm_stream_t stream);
 
 #ifdef __cplusplus
 }
