@@ -743,7 +743,7 @@ def main():
     ap.add_argument("--no-cpu", action="store_true", help="skip the cpu_baseline leg")
     ap.add_argument("--no-extras", action="store_true", help="only the headline step (for ncu runs)")
     ap.add_argument("--only-cfg5", action="store_true", help=argparse.SUPPRESS)
-    ap.add_argument("--arch", default=None, choices=["movolorn", "batasun", "fafelix", "nununex", "pekasun"],
+    ap.add_argument("--arch", default=None, choices=["movolorn", "batasun", "fafelix", "nununex", "pekasun", "fikudra"],
                     help="instead of the headline workload: prefill / decode throughput of this model design beside "
                          "the closest existing model at equal size, and its kernels against the measured peaks")
     ap.add_argument("--arch-sizes", default="1b-like,8b-like", help="with --arch: comma-separated size names")
@@ -759,6 +759,8 @@ def main():
             from compactor_vllm.benchmarks import nununex_compare as arch_compare
         elif args.arch == "pekasun":
             from compactor_vllm.benchmarks import pekasun_compare as arch_compare
+        elif args.arch == "fikudra":
+            from compactor_vllm.benchmarks import fikudra_compare as arch_compare
         else:
             from compactor_vllm.benchmarks import arch_compare
 
