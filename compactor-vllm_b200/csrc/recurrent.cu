@@ -921,44 +921,73 @@ __global__ void __launch_bounds__(MAXT) matrix_memory_kernel(const T* __restrict
 // ---------------------------------------------------------------------------------------------------------
 // Decays of the gated linear attention.  a [T, rank] (model type), w [channels, rank] (model type), bias [channels]:
 //   z = w a + bias (fp32 sums);  alpha = sigmoid(z)^(1 / tau) = exp(-softplus(-z) / tau),  fp32 [T, channels].
-// grid (channel blocks of 256, token tiles): a thread keeps its channel's weights (RANK at a time) in registers and
+// grid (channel blocks of 256, token tiles): a thread keeps its channel's weights (sixteen at a time) in registers and
 // walks the tile's tokens, whose inputs lie in shared memory.
 // ---------------------------------------------------------------------------------------------------------
 constexpr int kDecayRank = 16;     // weights in registers
 constexpr int kDecayTokens = 32;   // tokens per tile
 constexpr int kDecayMaxRank = 256;
 
+// sixteen weights of a channel from number r0 on (zeros past the rank)
+template <typename T>
+__device__ __forceinline__ void load_weights16(float (&w)[kDecayRank], const T* row, int r0, int rank, bool vec) {
+  if (vec && r0 + kDecayRank <= rank) {
+    constexpr int E = 16 / sizeof(T);
+#pragma unroll
+    for (int r = 0; r < kDecayRank; r += E) {
+      const uint4 t = *reinterpret_cast<const uint4*>(row + r0 + r);
+      const uint32_t x[4] = {t.x, t.y, t.z, t.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        if constexpr (sizeof(T) == 2) {
+          const float2 p = unpack2<true>(x[e]);
+          w[r + 2 * e] = p.x;
+          w[r + 2 * e + 1] = p.y;
+        } else {
+          w[r + e] = __uint_as_float(x[e]);
+        }
+      }
+    }
+  } else {
+#pragma unroll
+    for (int r = 0; r < kDecayRank; ++r) w[r] = r0 + r < rank ? to_f<T>(row[r0 + r]) : 0.f;
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) lowrank_decay_kernel(const T* __restrict__ a, int64_t a_stride,
                                                             const T* __restrict__ w, const float* __restrict__ bias,
                                                             float inv_tau, float* __restrict__ alpha,
-                                                            int64_t alpha_stride, int tokens, int channels, int rank) {
-  __shared__ __align__(16) float sa[kDecayTokens][kDecayMaxRank];
+                                                            int64_t alpha_stride, int tokens, int channels, int rank,
+                                                            int vec) {
+  extern __shared__ __align__(16) float sa[];       // [kDecayTokens][padded]
   const int t0 = blockIdx.y * kDecayTokens, n = min(kDecayTokens, tokens - t0);
   const int padded = (rank + kDecayRank - 1) / kDecayRank * kDecayRank;
   for (int i = threadIdx.x; i < n * padded; i += 256) {
     const int t = i / padded, r = i - t * padded;
-    sa[t][r] = r < rank ? to_f<T>(a[(int64_t)(t0 + t) * a_stride + r]) : 0.f;
+    sa[i] = r < rank ? to_f<T>(a[(int64_t)(t0 + t) * a_stride + r]) : 0.f;
   }
   __syncthreads();
   const int c = blockIdx.x * 256 + threadIdx.x;
   if (c >= channels) return;
   const T* wr = w + (int64_t)c * rank;
   const float b = bias[c];
-  for (int g = 0; g < n; g += 8) {
-    float z[8];
+  float wv[kDecayRank];
+  load_weights16<T>(wv, wr, 0, rank, vec);
+  constexpr int G = 4;      // tokens side by side
+  for (int g = 0; g < n; g += G) {
+    float z[G];
 #pragma unroll
-    for (int k = 0; k < 8; ++k) z[k] = b;
-    for (int r0 = 0; r0 < rank; r0 += kDecayRank) {
-      float wv[kDecayRank];
+    for (int k = 0; k < G; ++k) z[k] = b;
+    for (int r0 = 0; r0 < padded; r0 += kDecayRank) {
+      if (padded > kDecayRank) load_weights16<T>(wv, wr, r0, rank, vec);
 #pragma unroll
-      for (int r = 0; r < kDecayRank; ++r) wv[r] = r0 + r < rank ? to_f<T>(wr[r0 + r]) : 0.f;
-#pragma unroll
-      for (int k = 0; k < 8; ++k)
+      for (int k = 0; k < G; ++k)
         if (g + k < n) {
+          const float* row = sa + (g + k) * padded + r0;
 #pragma unroll
           for (int r = 0; r < kDecayRank; r += 4) {
-            const float4 x = *reinterpret_cast<const float4*>(&sa[g + k][r0 + r]);
+            const float4 x = *reinterpret_cast<const float4*>(row + r);
             z[k] = fmaf(wv[r], x.x, z[k]);
             z[k] = fmaf(wv[r + 1], x.y, z[k]);
             z[k] = fmaf(wv[r + 2], x.z, z[k]);
@@ -967,9 +996,9 @@ __global__ void __launch_bounds__(256) lowrank_decay_kernel(const T* __restrict_
         }
     }
 #pragma unroll
-    for (int k = 0; k < 8; ++k)
+    for (int k = 0; k < G; ++k)
       if (g + k < n) {
-        const float soft = z[k] < -20.f ? -z[k] : log1pf(expf(-z[k]));      // softplus(-z)
+        const float soft = fmaxf(-z[k], 0.f) + log1pf(expf(-fabsf(z[k])));             // softplus(-z)
         alpha[(int64_t)(t0 + g + k) * alpha_stride + c] = exp_1ulp(-soft * inv_tau);   // multiplies the state token after token
       }
   }
@@ -979,32 +1008,18 @@ __global__ void __launch_bounds__(256) lowrank_decay_kernel(const T* __restrict_
 // Gated linear attention.  q, k (H x D), v and the gate (H x Dv) are columns of proj (model type) at q_off, k_off (+ h * D),
 // v_off, gate_off (+ h * Dv); alpha [T, H * D] fp32.  Per head  S <- diag(alpha) S + k v^T,  o = q_scale S^T q.
 //
-// Nothing of a token waits for another token's read-out, so a thread keeps a TILE of the state: 8 rows x C value columns
-// (KS lanes of a warp hold the key rows of C columns, KS * 8 >= D; rows beyond D stay zero), and every key-sized number it
-// fetches serves C columns.  A lane's rows are two runs of four, ks * 4 and KS * 4 + ks * 4 onwards, so that neighbouring
-// lanes read neighbouring 16 bytes.  Inputs are staged as they are stored, `tok` tokens at a time, two stages deep: the
-// next stage is on its way (cp.async; plain loads where rows are not 16-byte multiples) while this one runs.  A token's
-// numbers are fetched one token ahead, and the sums over the key lanes of a token's C outputs run while the next token's
-// products do: each exchange halves the columns a lane is left with until one remains.
+// A thread keeps a TILE of the state: 8 rows x C value columns (KS lanes of a warp hold the key rows of C columns,
+// KS * 8 >= D; rows beyond D stay zero), so every key-sized number it fetches serves C columns.  A lane's rows are two runs
+// of four, ks * 4 and KS * 4 + ks * 4 onwards, so that neighbouring lanes read neighbouring 16 bytes.
+//
+// Tokens are taken in blocks of U.  With S the state before a block and its tokens counted 0 .. U - 1,
+//   o_t = (q_t alpha_0 .. alpha_t) . S + sum_(s <= t) p_ts v_s,     p_ts = q_t . (alpha_(s+1) .. alpha_t k_s)
+//   S  <- diag(alpha_0 .. alpha_(U-1)) S + sum_s (alpha_(s+1) .. alpha_(U-1) k_s) v_s^T
+// - the numbers of the recurrence with products of decays (never quotients) made once per CTA, per stage of `tok` tokens,
+// by a warp per block; the state then takes one multiplication per block and two fused ones per token, and the read-outs
+// of a block do not wait for one another.  The next stage's inputs arrive (cp.async; plain loads where rows are not
+// 16-byte multiples) while the state's products run.
 // ---------------------------------------------------------------------------------------------------------
-// four numbers as they are stored; turned into floats where they are used
-template <typename T>
-struct Quad;
-template <>
-struct Quad<float> {
-  float4 v;
-  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float4*>(p); }
-  __device__ __forceinline__ float2 lo() const { return make_float2(v.x, v.y); }
-  __device__ __forceinline__ float2 hi() const { return make_float2(v.z, v.w); }
-};
-template <>
-struct Quad<__nv_bfloat16> {
-  uint2 v;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint2*>(p); }
-  __device__ __forceinline__ float2 lo() const { return unpack2<true>(v.x); }
-  __device__ __forceinline__ float2 hi() const { return unpack2<true>(v.y); }
-};
-
 __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
   const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
@@ -1012,6 +1027,7 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src) {
 
 constexpr int kGlaTok = 32;     // most tokens staged at a time
 constexpr int kGlaRows = 8;     // state rows per thread
+constexpr int kGlaBlock = 4;    // tokens per block (single-token steps: 1)
 
 struct GlaArgs {
   int q_off, k_off, v_off;
@@ -1021,6 +1037,7 @@ struct GlaArgs {
   float q_scale;
   int vec_key, vec_val;   // key- / value-sized rows move as 16-byte pieces
   int CP;                 // staged value row: CW rounded up to 8
+  int out_pairs;          // 16-bit outputs are written two columns at a time
 };
 
 // n rows of `len` numbers (row stride `stride`) -> shared rows of `pitch` numbers
@@ -1037,17 +1054,25 @@ __device__ __forceinline__ void stage_rows(T* dst, int pitch, const T* src, int6
   }
 }
 
-template <typename T, int KS, int C>
+template <typename T, int KS, int C, int U>
 __global__ void __launch_bounds__(512) gla_scan_kernel(const T* __restrict__ proj, GlaArgs ga, RecurArgs a) {
   namespace cg = cooperative_groups;
-  constexpr int DP = KS * kGlaRows;
+  constexpr int DP = KS * kGlaRows, NV = U * C;
   extern __shared__ __align__(16) unsigned char smraw[];
   const int D = a.D, Dv = a.Dv, CW = a.CW, CP = ga.CP, tok = a.tok;
-  // one stage: alpha [tok][DP] fp32, q, k [tok][DP], v, gate [tok][CP]; two of them, then the outputs and the sums
-  const int stage_bytes = tok * (DP * 4 + (2 * DP + 2 * CP) * (int)sizeof(T));
-  float* so = reinterpret_cast<float*>(smraw + 2 * stage_bytes);   // [tok][CW]
-  float* part = so + tok * CW;                                     // [2][kGlaTok]
-  float* sinv = part + 2 * kGlaTok;                                // [kGlaTok]
+  // a stage as it arrives (consumed by the transform, then free for the next stage's loads)
+  float* al = reinterpret_cast<float*>(smraw);            // [tok][DP] alpha
+  T* rq = reinterpret_cast<T*>(al + tok * DP);            // [tok][DP]
+  T* rk = rq + tok * DP;                                  // [tok][DP]
+  T* vg = rk + tok * DP;                                  // [2 stages][v, gate][tok][CP]
+  // ... and as the state's products read it
+  float* tq = reinterpret_cast<float*>(vg + 4 * tok * CP);   // [tok][DP]
+  float* tk = tq + tok * DP;                              // [tok][DP]
+  float* ta = tk + tok * DP;                              // [tok / U][DP]
+  float* tp = ta + tok / U * DP;                          // [tok / U][U][U]
+  float* so = tp + tok * U;                               // [tok][CW] outputs
+  float* part = so + tok * CW;                            // [2][kGlaTok]
+  float* sinv = part + 2 * kGlaTok;                       // [kGlaTok]
   const int h = blockIdx.x / a.VT, vt = blockIdx.x % a.VT, b = blockIdx.y;
   int t0, n_new, start;
   portion(a.g, b, t0, n_new, start);
@@ -1059,6 +1084,21 @@ __global__ void __launch_bounds__(512) gla_scan_kernel(const T* __restrict__ pro
   const int col0 = grp * C;             // this thread's first column (of the CTA's)
   const bool live = col0 < ncol;
 
+  auto issue = [&](int j0, int buf) {
+    const int n = min(tok, n_new - j0);
+    T *sv = vg + buf * 2 * tok * CP, *sg = sv + tok * CP;
+    const T* row = proj + (int64_t)(t0 + j0) * ga.proj_stride;
+    stage_rows<float>(al, DP, ga.alpha + (int64_t)(t0 + j0) * ga.alpha_stride + h * D, ga.alpha_stride, D, n, ga.vec_key);
+    stage_rows<T>(rq, DP, row + ga.q_off + h * D, ga.proj_stride, D, n, ga.vec_key);
+    stage_rows<T>(rk, DP, row + ga.k_off + h * D, ga.proj_stride, D, n, ga.vec_key);
+    stage_rows<T>(sv, CP, row + ga.v_off + h * Dv + c0, ga.proj_stride, ncol, n, ga.vec_val);
+    stage_rows<T>(sg, CP, static_cast<const T*>(a.gate) + (int64_t)(t0 + j0) * a.gate_stride + a.gate_off + h * Dv + c0,
+                  a.gate_stride, ncol, n, ga.vec_val);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    // the last block's missing tokens: their keys are zero, and so must their values be (0 * garbage)
+    for (int i = n * CP + tid; i < (n + U - 1) / U * U * CP; i += blockDim.x) sv[i] = from_f<T>(0.f);
+  };
+  issue(0, 0);
   // state tile: S[j][r] = rows (2 r, 2 r + 1 of the thread's eight) of column col0 + j
   float2 S[C][kGlaRows / 2];
   {
@@ -1086,119 +1126,171 @@ __global__ void __launch_bounds__(512) gla_scan_kernel(const T* __restrict__ pro
       }
     }
   }
-  if (D != DP || ncol != CP) {   // pads: keys, queries and decays beyond D, values beyond the columns
-    for (int i = tid; i < 2 * stage_bytes / 16; i += blockDim.x)
-      reinterpret_cast<uint4*>(smraw)[i] = make_uint4(0u, 0u, 0u, 0u);
-    __syncthreads();
-  }
-  auto issue = [&](int j0, int buf) {
-    const int n = min(tok, n_new - j0);
-    unsigned char* base = smraw + buf * stage_bytes;
-    float* al = reinterpret_cast<float*>(base);
-    T* sq = reinterpret_cast<T*>(al + tok * DP);
-    T *sk = sq + tok * DP, *sv = sk + tok * DP, *sg = sv + tok * CP;
-    const T* row = proj + (int64_t)(t0 + j0) * ga.proj_stride;
-    stage_rows<float>(al, DP, ga.alpha + (int64_t)(t0 + j0) * ga.alpha_stride + h * D, ga.alpha_stride, D, n, ga.vec_key);
-    stage_rows<T>(sq, DP, row + ga.q_off + h * D, ga.proj_stride, D, n, ga.vec_key);
-    stage_rows<T>(sk, DP, row + ga.k_off + h * D, ga.proj_stride, D, n, ga.vec_key);
-    stage_rows<T>(sv, CP, row + ga.v_off + h * Dv + c0, ga.proj_stride, ncol, n, ga.vec_val);
-    stage_rows<T>(sg, CP, static_cast<const T*>(a.gate) + (int64_t)(t0 + j0) * a.gate_stride + a.gate_off + h * Dv + c0,
-                  a.gate_stride, ncol, n, ga.vec_val);
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  issue(0, 0);
+  if (D != DP)   // rows beyond D: zero keys, queries and decays, written once
+    for (int i = tid; i < (2 * tok + tok / U) * DP; i += blockDim.x) tq[i] = 0.f;
   int stage = 0;
   for (int j0 = 0; j0 < n_new; j0 += tok, ++stage) {
-    const int n = min(tok, n_new - j0);
-    if (j0 + tok < n_new) {
-      issue(j0 + tok, (stage + 1) & 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
+    const int n = min(tok, n_new - j0), blocks = (n + U - 1) / U;
+    const T *sv = vg + (stage & 1) * 2 * tok * CP, *sg = sv + tok * CP;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const unsigned char* base = smraw + (stage & 1) * stage_bytes;
-    const float* al = reinterpret_cast<const float*>(base);
-    const T* sq = reinterpret_cast<const T*>(al + tok * DP);
-    const T *sk = sq + tok * DP, *sv = sk + tok * DP, *sg = sv + tok * CP;
-    {
-      const int at = ks * 4, vat = live ? col0 : 0;
-      Quad<float> na[2];
-      Quad<T> nq[2], nk[2];
-      float nv[C], pend[C];
-      auto fetch = [&](int c) {
+    // a warp per block of U tokens, a lane per key channel
+    for (int blk = warp; blk < blocks; blk += warps) {
+      float pp[U * U];
 #pragma unroll
-        for (int q4 = 0; q4 < 2; ++q4) {
-          na[q4].load(al + c * DP + q4 * KS * 4 + at);
-          nq[q4].load(sq + c * DP + q4 * KS * 4 + at);
-          nk[q4].load(sk + c * DP + q4 * KS * 4 + at);
+      for (int i = 0; i < U * U; ++i) pp[i] = 0.f;
+      for (int d = lane; d < D; d += 32) {
+        float q[U], k[U], f[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const bool on = U == 1 || blk * U + u < n;
+          const int at = (blk * U + u) * DP + d;
+          q[u] = on ? to_f<T>(rq[at]) : 0.f;
+          k[u] = on ? to_f<T>(rk[at]) : 0.f;
+          f[u] = on ? al[at] : 1.f;
+        }
+        float w = 1.f;
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          w *= f[u];
+          tq[(blk * U + u) * DP + d] = q[u] * w;
+        }
+        ta[blk * DP + d] = w;
+        w = 1.f;
+#pragma unroll
+        for (int u = U - 1; u >= 0; --u) {
+          tk[(blk * U + u) * DP + d] = k[u] * w;
+          w *= f[u];
         }
 #pragma unroll
-        for (int j = 0; j < C; ++j) nv[j] = to_f<T>(sv[c * CP + vat + j]);
-      };
-      // sums of a token's C partial outputs over the KS key lanes; a lane ends up with C / min(C, KS) columns from `first`
-      auto finish = [&](int c) {
-        int left = C, first = 0;
+        for (int s = 0; s < U; ++s) {
+          float ks_ = k[s];
 #pragma unroll
-        for (int o = 1; o < KS; o <<= 1) {
+          for (int t = s; t < U; ++t) {
+            if (t > s) ks_ *= f[t];
+            pp[t * U + s] = fmaf(q[t], ks_, pp[t * U + s]);
+          }
+        }
+      }
+      if constexpr (U == 1) {
+        pp[0] = warp_sum(pp[0]);
+        if (lane == 0) tp[blk] = pp[0];
+      } else {   // U * U <= 32 sums over the lanes: each exchange halves what a lane is left with
+        int left = U * U, first = 0;
+#pragma unroll
+        for (int d = 1; d < 32; d <<= 1) {
           if (left > 1) {
-            const bool up = (ks & o) != 0;
+            const bool up = (lane & d) != 0;
             left >>= 1;
 #pragma unroll
-            for (int j = 0; j < C / 2; ++j)
+            for (int j = 0; j < U * U / 2; ++j)
               if (j < left) {
-                const float send = up ? pend[j] : pend[j + left], keep = up ? pend[j + left] : pend[j];
-                pend[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                const float send = up ? pp[j] : pp[j + left], keep = up ? pp[j + left] : pp[j];
+                pp[j] = keep + __shfl_xor_sync(0xffffffffu, send, d);
               }
             if (up) first += left;
           } else {
-            pend[0] += __shfl_xor_sync(0xffffffffu, pend[0], o);
+            pp[0] += __shfl_xor_sync(0xffffffffu, pp[0], d);
           }
         }
-        if (ks < C) {
-#pragma unroll
-          for (int j = 0; j < C; ++j)
-            if (j < left && col0 + first + j < ncol) so[c * CW + col0 + first + j] = pend[j] * ga.q_scale;
-        }
-      };
-      fetch(0);
-      for (int c = 0; c < n; ++c) {
-        float2 ac[4], qc[4], kc[4];
-        float vc[C], op_s[C];
-#pragma unroll
-        for (int q4 = 0; q4 < 2; ++q4) {
-          ac[2 * q4] = na[q4].lo(), ac[2 * q4 + 1] = na[q4].hi();
-          qc[2 * q4] = nq[q4].lo(), qc[2 * q4 + 1] = nq[q4].hi();
-          kc[2 * q4] = nk[q4].lo(), kc[2 * q4 + 1] = nk[q4].hi();
-        }
-#pragma unroll
-        for (int j = 0; j < C; ++j) vc[j] = nv[j];
-        if (c + 1 < n) fetch(c + 1);
-        if (c > 0) finish(c - 1);
-#pragma unroll
-        for (int j = 0; j < C; ++j) {
-          const float2 v2 = make_float2(vc[j], vc[j]);
-          float2 o2 = make_float2(0.f, 0.f);
-#pragma unroll
-          for (int r = 0; r < 4; ++r) {
-            S[j][r] = __ffma2_rn(ac[r], S[j][r], __fmul2_rn(kc[r], v2));
-            o2 = __ffma2_rn(qc[r], S[j][r], o2);
-          }
-          op_s[j] = o2.x + o2.y;
-        }
-#pragma unroll
-        for (int j = 0; j < C; ++j) pend[j] = op_s[j];
+        if (lane < U * U) tp[blk * U * U + first] = pp[0];
       }
-      finish(n - 1);
     }
     __syncthreads();
-    // unit norm over ALL Dv columns of the head (the cluster's CTAs exchange their sums of squares), weight, gate
+    if (j0 + tok < n_new) issue(j0 + tok, (stage + 1) & 1);
+    {
+      const int at = ks * 4, vat = live ? col0 : 0;
+      for (int blk = 0; blk < blocks; ++blk) {
+        const int c = blk * U;
+        float o[NV];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {   // what the tokens read of the state before the block
+          const float4 q0 = *reinterpret_cast<const float4*>(tq + (c + u) * DP + at);
+          const float4 q1 = *reinterpret_cast<const float4*>(tq + (c + u) * DP + KS * 4 + at);
+          float2 o2[C];
+#pragma unroll
+          for (int j = 0; j < C; ++j) o2[j] = __fmul2_rn(make_float2(q0.x, q0.y), S[j][0]);
+#pragma unroll
+          for (int j = 0; j < C; ++j) o2[j] = __ffma2_rn(make_float2(q0.z, q0.w), S[j][1], o2[j]);
+#pragma unroll
+          for (int j = 0; j < C; ++j) o2[j] = __ffma2_rn(make_float2(q1.x, q1.y), S[j][2], o2[j]);
+#pragma unroll
+          for (int j = 0; j < C; ++j) o2[j] = __ffma2_rn(make_float2(q1.z, q1.w), S[j][3], o2[j]);
+#pragma unroll
+          for (int j = 0; j < C; ++j) o[u * C + j] = o2[j].x + o2[j].y;
+        }
+        {
+          const float4 a0 = *reinterpret_cast<const float4*>(ta + blk * DP + at);
+          const float4 a1 = *reinterpret_cast<const float4*>(ta + blk * DP + KS * 4 + at);
+#pragma unroll
+          for (int j = 0; j < C; ++j) {
+            S[j][0] = __fmul2_rn(make_float2(a0.x, a0.y), S[j][0]);
+            S[j][1] = __fmul2_rn(make_float2(a0.z, a0.w), S[j][1]);
+            S[j][2] = __fmul2_rn(make_float2(a1.x, a1.y), S[j][2]);
+            S[j][3] = __fmul2_rn(make_float2(a1.z, a1.w), S[j][3]);
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const float4 k0 = *reinterpret_cast<const float4*>(tk + (c + u) * DP + at);
+          const float4 k1 = *reinterpret_cast<const float4*>(tk + (c + u) * DP + KS * 4 + at);
+#pragma unroll
+          for (int j = 0; j < C; ++j) {
+            const float v = to_f<T>(sv[(c + u) * CP + vat + j]);
+            const float2 v2 = make_float2(v, v);
+            S[j][0] = __ffma2_rn(make_float2(k0.x, k0.y), v2, S[j][0]);
+            S[j][1] = __ffma2_rn(make_float2(k0.z, k0.w), v2, S[j][1]);
+            S[j][2] = __ffma2_rn(make_float2(k1.x, k1.y), v2, S[j][2]);
+            S[j][3] = __ffma2_rn(make_float2(k1.z, k1.w), v2, S[j][3]);
+          }
+        }
+        // sums over the key lanes of all U * C outputs together, halving as above; the lane a sum ends up with adds what
+        // the token reads of the block itself
+        int left = NV, first = 0;
+#pragma unroll
+        for (int d = 1; d < KS; d <<= 1) {
+          if (left > 1) {
+            const bool up = (ks & d) != 0;
+            left >>= 1;
+#pragma unroll
+            for (int j = 0; j < NV / 2; ++j)
+              if (j < left) {
+                const float send = up ? o[j] : o[j + left], keep = up ? o[j + left] : o[j];
+                o[j] = keep + __shfl_xor_sync(0xffffffffu, send, d);
+              }
+            if (up) first += left;
+          } else {
+            o[0] += __shfl_xor_sync(0xffffffffu, o[0], d);
+          }
+        }
+        if (KS <= NV || ks < NV) {
+#pragma unroll
+          for (int j = 0; j < NV; ++j)
+            if (j < left) {
+              const int u = (first + j) / C, col = col0 + (first + j) % C;
+              if (col < ncol) {
+                float acc = o[j];
+#pragma unroll
+                for (int s = 0; s < U; ++s)
+                  acc = fmaf(tp[blk * U * U + u * U + s], to_f<T>(sv[(c + s) * CP + col]), acc);
+                so[(c + u) * CW + col] = acc * ga.q_scale;
+              }
+            }
+        }
+      }
+    }
+    __syncthreads();
+    // unit norm over ALL Dv columns of the head (the cluster's CTAs exchange their sums of squares), weight, gate;
+    // eight lanes per token
     float* mine = part + (stage & 1) * kGlaTok;
-    for (int c = warp; c < n; c += warps) {
+    for (int cb = warp * 4; cb < n; cb += warps * 4) {
+      const int c = cb + (lane >> 3);
       float ss = 0.f;
-      for (int j = lane; j < ncol; j += 32) ss = fmaf(so[c * CW + j], so[c * CW + j], ss);
-      ss = warp_sum(ss);
-      if (lane == 0) mine[c] = ss;
+      if (c < n)
+        for (int j = lane & 7; j < ncol; j += 8) ss = fmaf(so[c * CW + j], so[c * CW + j], ss);
+#pragma unroll
+      for (int d = 4; d > 0; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+      if ((lane & 7) == 0 && c < n) mine[c] = ss;
     }
     if (a.VT > 1) cg::this_cluster().sync();
     else __syncthreads();
@@ -1215,13 +1307,20 @@ __global__ void __launch_bounds__(512) gla_scan_kernel(const T* __restrict__ pro
     __syncthreads();
     if (ncol > 0) {
       T* out = static_cast<T*>(a.out);
-      TileWalk w(ncol);
-      for (; w.c < n; w.next()) {
-        const float gz = to_f<T>(sg[w.c * CP + w.d]);
-        const int col = c0 + w.d;
-        out[(int64_t)(t0 + j0 + w.c) * a.out_stride + h * Dv + col] =
-            from_f<T>(so[w.c * CW + w.d] * sinv[w.c] * a.norm_w[h * a.norm_head_stride + col] *
-                      (a.gate_kind ? sigmoid_f(gz) : silu_f(gz)));
+      auto value = [&](int c, int j) {
+        const float gz = to_f<T>(sg[c * CP + j]);
+        return so[c * CW + j] * sinv[c] * a.norm_w[h * a.norm_head_stride + c0 + j] *
+               (a.gate_kind ? sigmoid_f(gz) : silu_f(gz));
+      };
+      if (sizeof(T) == 2 && ga.out_pairs) {
+        TileWalk w(ncol / 2);
+        for (; w.c < n; w.next())
+          *reinterpret_cast<uint32_t*>(out + (int64_t)(t0 + j0 + w.c) * a.out_stride + h * Dv + c0 + 2 * w.d) =
+              pack2<true>(value(w.c, 2 * w.d), value(w.c, 2 * w.d + 1));
+      } else {
+        TileWalk w(ncol);
+        for (; w.c < n; w.next())
+          out[(int64_t)(t0 + j0 + w.c) * a.out_stride + h * Dv + c0 + w.d] = from_f<T>(value(w.c, w.d));
       }
     }
     __syncthreads();
@@ -1253,10 +1352,11 @@ __global__ void __launch_bounds__(512) gla_scan_kernel(const T* __restrict__ pro
 // CTA, VT CTAs (a cluster).  Warps work alone, so a portion wants about one per scheduler of the GPU: two columns per
 // thread instead of four while four would leave schedulers idle; CTAs of four warps, more when the step has CTAs enough.
 struct GlaShape {
-  int KS, C, VT, warps, CW, CP, tok;
+  int KS, C, U, VT, warps, CW, CP, tok;
   size_t smem(size_t elem) const {
-    return 2 * (size_t)tok * ((size_t)KS * kGlaRows * (4 + 2 * elem) + 2 * (size_t)CP * elem) +
-           sizeof(float) * ((size_t)tok * CW + 3 * kGlaTok);
+    const size_t DP = (size_t)KS * kGlaRows;
+    return tok * (DP * (4 + 2 * elem) + 4 * (size_t)CP * elem + 8 * DP + 4 * DP / U + 4 * U + 4 * (size_t)CW) +
+           sizeof(float) * 3 * kGlaTok;
   }
 };
 
@@ -1266,19 +1366,20 @@ inline GlaShape gla_shape(int D, int Dv, int64_t pairs, int max_new, size_t elem
   while (s.KS * kGlaRows < D) s.KS <<= 1;
   auto warps_of = [&](int C) { return cdiv(Dv, 32 / s.KS * C); };
   const int forced = test_options().gla_layout.load();   // 100 * VT + C (tests and measurements)
-  s.C = max_new > 1 && pairs * warps_of(4) < 4 * (int64_t)sm_count() ? 2 : 4;
-  if (forced > 0) s.C = forced % 100 == 2 ? 2 : 4;
+  s.C = max_new > 1 && pairs * warps_of(4) < 4 * (int64_t)sm_count() && warps_of(2) <= 64 ? 2 : 4;
+  if (forced > 0 && max_new > 1) s.C = forced % 100 == 2 ? 2 : 4;
   const int w = warps_of(s.C);
   s.VT = 1;
-  while (s.VT < 8 && s.VT * 4 < w) s.VT *= 2;
+  while (s.VT < 8 && s.VT * (max_new > 1 ? 8 : 16) < w) s.VT *= 2;
   while (s.VT > 1 && pairs * s.VT >= 4 * (int64_t)sm_count() && cdiv(w, s.VT / 2) <= 16) s.VT /= 2;
   if (forced > 0 && forced / 100 >= 1 && forced / 100 <= 8 && cdiv(w, forced / 100) <= 16) s.VT = forced / 100;
   s.warps = cdiv(w, s.VT);
   s.CW = s.warps * (32 / s.KS) * s.C;
   s.CP = cdiv(s.CW, 8) * 8;
-  s.tok = 1;
+  s.U = max_new > 1 ? kGlaBlock : 1;
+  s.tok = s.U;
   while (s.tok < kGlaTok && s.tok < max_new) s.tok <<= 1;
-  while (s.tok > 1 && s.smem(elem) > 96 * 1024) s.tok >>= 1;
+  while (s.tok > s.U && s.smem(elem) > 110 * 1024) s.tok >>= 1;
   return s;
 }
 
@@ -1375,11 +1476,11 @@ cudaError_t launch_clustered(K kern, dim3 grid, int threads, size_t smem, cudaSt
   return cudaLaunchKernelEx(&cfg, kern, args...);
 }
 
-template <typename T, int KS, int C>
+template <typename T, int KS, int C, int U>
 int launch_gla(const GlaShape& sh, dim3 grid, cudaStream_t st, const void* proj, const GlaArgs& ga, const RecurArgs& a) {
   static std::atomic<uint64_t> attr{0};
-  CVLLM_CHECK_CUDA(ensure_max_dyn_smem((const void*)gla_scan_kernel<T, KS, C>, 200 * 1024, attr));
-  CVLLM_CHECK_CUDA(launch_clustered(gla_scan_kernel<T, KS, C>, grid, sh.warps * 32, sh.smem(sizeof(T)), st, sh.VT,
+  CVLLM_CHECK_CUDA(ensure_max_dyn_smem((const void*)gla_scan_kernel<T, KS, C, U>, 200 * 1024, attr));
+  CVLLM_CHECK_CUDA(launch_clustered(gla_scan_kernel<T, KS, C, U>, grid, sh.warps * 32, sh.smem(sizeof(T)), st, sh.VT,
                                     static_cast<const T*>(proj), ga, a));
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
@@ -1388,7 +1489,9 @@ int launch_gla(const GlaShape& sh, dim3 grid, cudaStream_t st, const void* proj,
 template <typename T>
 int dispatch_gla(const GlaShape& sh, dim3 grid, cudaStream_t st, const void* proj, const GlaArgs& ga, const RecurArgs& a) {
 #define CVLLM_GLA(KK) \
-  return sh.C == 2 ? launch_gla<T, KK, 2>(sh, grid, st, proj, ga, a) : launch_gla<T, KK, 4>(sh, grid, st, proj, ga, a)
+  return sh.U == 1 ? launch_gla<T, KK, 4, 1>(sh, grid, st, proj, ga, a)                \
+         : sh.C == 2 ? launch_gla<T, KK, 2, kGlaBlock>(sh, grid, st, proj, ga, a)      \
+                     : launch_gla<T, KK, 4, kGlaBlock>(sh, grid, st, proj, ga, a)
   switch (sh.KS) {
     case 1: CVLLM_GLA(1);
     case 2: CVLLM_GLA(2);
@@ -1641,14 +1744,16 @@ extern "C" int cvllm_lowrank_decay(const void* a, int64_t a_stride, const void* 
   CVLLM_CHECK_SUPPORTED(rank <= kDecayMaxRank && cdiv(tokens, kDecayTokens) <= 65535);
   auto st = static_cast<cudaStream_t>(stream);
   const dim3 grid(cdiv(channels, 256), cdiv(tokens, kDecayTokens));
+  const size_t smem = sizeof(float) * kDecayTokens * (size_t)(cdiv(rank, kDecayRank) * kDecayRank);   // <= 32 KB
+  const int vec = rank % (dtype == CVLLM_BF16 ? 8 : 4) == 0 && aligned16(w);
   if (dtype == CVLLM_BF16)
-    lowrank_decay_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(static_cast<const __nv_bfloat16*>(a), a_stride,
-                                                              static_cast<const __nv_bfloat16*>(w), bias, inv_tau, alpha,
-                                                              alpha_stride, tokens, channels, rank);
+    lowrank_decay_kernel<__nv_bfloat16><<<grid, 256, smem, st>>>(static_cast<const __nv_bfloat16*>(a), a_stride,
+                                                                 static_cast<const __nv_bfloat16*>(w), bias, inv_tau,
+                                                                 alpha, alpha_stride, tokens, channels, rank, vec);
   else
-    lowrank_decay_kernel<float><<<grid, 256, 0, st>>>(static_cast<const float*>(a), a_stride,
-                                                      static_cast<const float*>(w), bias, inv_tau, alpha, alpha_stride,
-                                                      tokens, channels, rank);
+    lowrank_decay_kernel<float><<<grid, 256, smem, st>>>(static_cast<const float*>(a), a_stride,
+                                                         static_cast<const float*>(w), bias, inv_tau, alpha,
+                                                         alpha_stride, tokens, channels, rank, vec);
   CVLLM_CHECK_LAUNCH();
   return CVLLM_OK;
 }
@@ -1674,7 +1779,8 @@ extern "C" int cvllm_gla_scan(const void* proj, int64_t proj_stride, int q_off, 
   const int vec_key = rows16 && D % E == 0 && q_off % E == 0 && k_off % E == 0 && aligned16(alpha) &&
                       alpha_stride % 4 == 0;
   const int vec_val = rows16 && Dv % E == 0 && sh.CW % E == 0 && v_off % E == 0 && gate_off % E == 0;
-  const GlaArgs ga{q_off, k_off, v_off, proj_stride, alpha, alpha_stride, q_scale, vec_key, vec_val, sh.CP};
+  const int out_pairs = Dv % 2 == 0 && sh.CW % 2 == 0 && out_stride % 2 == 0 && reinterpret_cast<uintptr_t>(out) % 4 == 0;
+  const GlaArgs ga{q_off, k_off, v_off, proj_stride, alpha, alpha_stride, q_scale, vec_key, vec_val, sh.CP, out_pairs};
   const RecurArgs a{{cu_seqlens_q, seq_start, positions, batch_mapping}, state, proj, proj_stride, gate_off, norm_w,
                     norm_head_stride, eps, out, out_stride, H, D, Dv, reserved_slot, sh.KS, sh.VT, sh.CW, sh.tok,
                     gate_kind};
